@@ -47,12 +47,16 @@ constexpr size_t SMEM_FLOATS = (size_t)QT * QS + (size_t)KC * KS + (size_t)KC * 
 //   value_in_key     the value of a key is its own first VD channels; the cache holds keys only
 //   slopes           a linear distance bias: slopes[h] * (query position - key position) is taken off the score of
 //                    query head h, after scale and cap (null: none)
+//   bias             a learned distance bias: bias[h * bias_len + min(query position - key position, bias_len - 1)] is
+//                    added to the score of query head h, after scale and cap (null: none)
 struct Extra {
     float softcap;
     const float* sink_values;
     int maps;
     int value_in_key;
     const float* slopes;
+    const float* bias;
+    int bias_len;
 };
 
 // key head and value head of query head h
@@ -111,6 +115,7 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ o
     // (with sink values: a term exp(sink_h) instead, so the maximum starts at sink_h)
     float m = sink ? (ex.sink_values ? ex.sink_values[h] : 0.f) : -INFINITY, l = sink ? 1.f : 0.f;
     const float slope = ex.slopes ? ex.slopes[h] : 0.f;
+    const float* bias = ex.bias ? ex.bias + (size_t)h * ex.bias_len : nullptr;
     float acc[NACC];
 #pragma unroll
     for (int i = 0; i < NACC; ++i) acc[i] = 0.f;
@@ -157,6 +162,7 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ o
             float sc = dot * scale;
             if (ex.softcap > 0.f) sc = ex.softcap * tanhf(sc / ex.softcap);
             if (ex.slopes) sc -= slope * (float)(p_row - key);
+            if (bias && seen) sc += bias[min(p_row - key, ex.bias_len - 1)];
             s[c] = seen ? sc : -INFINITY;
             cmax = fmaxf(cmax, s[c]);
         }
@@ -341,6 +347,7 @@ attention_single_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ 
                     float x = s[g] * scale;
                     if (ex.softcap > 0.f) x = ex.softcap * tanhf(x / ex.softcap);
                     if (ex.slopes) x -= ex.slopes[head0 + g * head_step] * (float)(p_query - key);
+                    if (ex.bias) x += ex.bias[(size_t)(head0 + g * head_step) * ex.bias_len + min(p_query - key, ex.bias_len - 1)];
                     sc[g * SK + kk] = x;
                 }
         }
@@ -572,9 +579,10 @@ RI_API int ri_attention_plain_ex(const void* q, int q_stride, void* out, int out
                                  const int* tile_q0, int n_tiles, int Hq, int Hkv, int page_size,
                                  float scale, int window, int block, int sink, float softcap,
                                  const float* sink_values, int maps, int value_in_key, int out_f32, const float* slopes,
-                                 void* stream) {
+                                 const float* bias, int bias_len, void* stream) {
     if (n_tiles <= 0) return 0;
-    const Extra ex{softcap, sink_values, maps, value_in_key, slopes};
+    const Extra ex{softcap, sink_values, maps, value_in_key, slopes, bias, bias_len};
+    if (bias && bias_len <= 0) return (int)cudaErrorInvalidValue;
     if (!extra_fits(Hq, Hkv, ex)) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == RI_BF16 && out_f32)
@@ -594,7 +602,7 @@ RI_API int ri_attention_plain(const void* q, int q_stride, void* out, int out_st
                               float scale, int window, int block, int sink, void* stream) {
     return ri_attention_plain_ex(q, q_stride, out, out_stride, cache, dtype, block_table, table_stride, cu_q, kv_len,
                                  tile_entry, tile_q0, n_tiles, Hq, Hkv, page_size, scale, window, block, sink,
-                                 0.f, nullptr, 1, 0, 0, nullptr, stream);
+                                 0.f, nullptr, 1, 0, 0, nullptr, nullptr, 0, stream);
 }
 
 // Entries that bring a single token (entry_list[i], -1: skip): keys and values of a kv head are read once
@@ -606,9 +614,10 @@ RI_API int ri_attention_single_ex(const void* q, int q_stride, void* out, int ou
                                   const int* entry_list, int n_entries, int Hq, int Hkv, int page_size, float scale,
                                   int window, int block, int sink, int splits, float* part, float softcap,
                                   const float* sink_values, int maps, int value_in_key, int out_f32,
-                                  const float* slopes, void* stream) {
+                                  const float* slopes, const float* bias, int bias_len, void* stream) {
     if (n_entries <= 0) return 0;
-    const Extra ex{softcap, sink_values, maps, value_in_key, slopes};
+    const Extra ex{softcap, sink_values, maps, value_in_key, slopes, bias, bias_len};
+    if (bias && bias_len <= 0) return (int)cudaErrorInvalidValue;
     if (!extra_fits(Hq, Hkv, ex)) return (int)cudaErrorInvalidValue;
     if (Hq / (Hkv * maps) > SG || SV > 4) return (int)cudaErrorNotSupported;
     if (splits < 1 || splits > 64 || (splits > 1 && !part)) return (int)cudaErrorInvalidValue;
@@ -643,7 +652,7 @@ RI_API int ri_attention_single(const void* q, int q_stride, void* out, int out_s
                                int window, int block, int sink, int splits, float* part, void* stream) {
     return ri_attention_single_ex(q, q_stride, out, out_stride, cache, dtype, block_table, table_stride, cu_q, kv_len,
                                   entry_list, n_entries, Hq, Hkv, page_size, scale, window, block, sink, splits, part,
-                                  0.f, nullptr, 1, 0, 0, nullptr, stream);
+                                  0.f, nullptr, 1, 0, 0, nullptr, nullptr, 0, stream);
 }
 
 RI_API int ri_attention_single_supports(int Hq, int Hkv) {

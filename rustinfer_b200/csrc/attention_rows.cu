@@ -83,6 +83,9 @@ struct Geometry {
     int splits;            // ranges the key tiles of a CTA are cut into (grid z); > 1: results go through `part`
     float scale, softcap;  // softcap 0: scores are not capped
     const float* slopes;   // slopes[h] * (query position - key position) is taken off head h's scores (null: no such bias)
+    const float* bias;     // bias[h * bias_len + min(query position - key position, bias_len - 1)] is added to head h's scores (null: none)
+    int bias_len;
+    int block;             // > 0: a query sees only keys of its own block of that many positions (counted from 0)
 };
 
 // keys k0 .. k0+KT-1 of key head `kh` (and, unless the values lie inside the keys, the values of value head `g`)
@@ -148,7 +151,8 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
     }
 
     const int p_first = pos0 + tok0, p_last = p_first + ntok - 1;
-    const int lo_tile = gm.window > 0 ? max(0, p_first - gm.window + 1) : 0;
+    int lo_tile = gm.window > 0 ? max(0, p_first - gm.window + 1) : 0;
+    if (gm.block > 0) lo_tile = max(lo_tile, p_first / gm.block * gm.block);
     int t_begin = lo_tile / KT, t_end = p_last / KT + 1;
     if (gm.splits > 1) {
         // this CTA's range of the key tiles; it may be empty
@@ -170,14 +174,17 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
     int p_row[2], lo_row[2];
     bool ok_row[2];
     float m[2], l[2] = {0.f, 0.f}, slope[2] = {0.f, 0.f};
+    const float* bias[2] = {nullptr, nullptr};
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         const int r = warp * 16 + (lane >> 2) + 8 * i;
         const int jj = r / Gc, hh = r - jj * Gc;
         ok_row[i] = jj < ntok && hh < nheads;
         if (gm.slopes && ok_row[i]) slope[i] = gm.slopes[head_of(hh)];
+        if (gm.bias) bias[i] = gm.bias + (size_t)(ok_row[i] ? head_of(hh) : 0) * gm.bias_len;
         p_row[i] = p_first + jj;
         lo_row[i] = gm.window > 0 ? max(0, p_row[i] - gm.window + 1) : 0;
+        if (gm.block > 0) lo_row[i] = max(lo_row[i], p_row[i] / gm.block * gm.block);
         m[i] = -INFINITY;
         if (gm.sink && gm.splits == 1 && ok_row[i]) {           // with ranges, the join adds the term once
             // a term exp(sink_h) without a value: the maximum starts there and, in the one lane of four whose
@@ -240,6 +247,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
                     float sc = s[n][e] * gm.scale;
                     if (gm.softcap > 0.f) sc = gm.softcap * tanhf(sc / gm.softcap);
                     sc -= slope[i] * (float)(p_row[i] - key);
+                    if (gm.bias) sc += __ldg(bias[i] + max(0, min(p_row[i] - key, gm.bias_len - 1)));
                     const bool seen = ok_row[i] && key <= p_row[i] && key >= lo_row[i];
                     s[n][e] = seen ? sc * LOG2E : -INFINITY;
                     mx[i] = fmaxf(mx[i], s[n][e]);
@@ -472,13 +480,15 @@ RI_API int ri_attention_rows(const void* q, int q_stride, void* out, int out_str
                              const int* tile_entry, const int* tile_tok0, int n_tiles, int Hq, int Hkv, int page_size,
                              float scale, int window, int sink, float softcap, const float* sink_values, int maps,
                              int value_in_key, int out_f32, int splits, float* part, const float* slopes,
-                             void* stream) {
+                             const float* bias, int bias_len, int block, void* stream) {
     if (n_tiles <= 0) return 0;
+    if (bias && bias_len <= 0) return (int)cudaErrorInvalidValue;
     if (splits < 1 || splits > 64 || (splits > 1 && !part)) return (int)cudaErrorInvalidValue;
     const int gc = ri_attention_rows_heads_per_cta(Hq, Hkv, maps);
     if (gc <= 0 || (value_in_key && (maps != 1 || VD > HD)) || q_stride % 8) return (int)cudaErrorInvalidValue;
     const int G = Hq / (Hkv * maps);
-    Geometry gm{Hq, Hkv, maps, gc, (G + gc - 1) / gc, MT / gc, page_size, window, sink, splits, scale, softcap, slopes};
+    Geometry gm{Hq, Hkv, maps, gc, (G + gc - 1) / gc, MT / gc, page_size, window, sink, splits, scale, softcap, slopes,
+                bias, bias_len, block};
     cudaStream_t s = (cudaStream_t)stream;
 #define RI_ROWS_GO(TO, VIK) launch<TO, VIK>(q, q_stride, out, out_stride, cache, block_table, table_stride, cu_q, kv_len, \
                                             tile_entry, tile_tok0, n_tiles, sink_values, part, gm, s)

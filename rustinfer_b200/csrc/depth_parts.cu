@@ -168,26 +168,47 @@ __global__ void rms_sandwich_kernel(const float* __restrict__ h_in, int in_strid
 // ----------------------------------------------------------------------- short causal convolution with a state
 // With x'[t][c] = x[t][c] + in_bias[c] (in_bias null: 0):
 // y[t][c] = (residual ? x'[t][c] : 0) + bias[c] + sum_j w[c][j] * x'[t - taps + 1 + j][c] over the tokens of one
-// entry; the taps - 1 inputs before the entry's first token come from state[slot] ([taps - 1][C], oldest first;
+// entry (then silu when `silu`); the taps - 1 inputs before the entry's first token come from state[slot] ([taps - 1][C], oldest first;
 // zeros for a new request), and the entry's last taps - 1 inputs go back there.  A thread owns one channel of a
 // chunk of CONV_CHUNK tokens of one entry (their loads in flight at once); the thread of an entry's first chunk is the only one that reads or
 // writes the channel's state.
 constexpr int CONV_MAX_TAPS = 8, CONV_CHUNK = 8;
+
+// The H columns behind x's C channels as step sizes of a recurrence, made in the same launch:
+//   dt[t][h] = softplus(x[t][C + h] + bias[h]),  decay[t][h] = exp(-exp(a_log[h]) * dt[t][h])
+struct StepSizes {
+    const float* bias;           // [H]; H = 0: none
+    const float* a_log;          // [H]
+    float* dt;                   // [T][H]
+    float* decay;                // [T][H]
+    int H;
+};
 
 template <typename TI, typename TO>
 __global__ void short_conv_kernel(const TI* __restrict__ x, int x_stride, const float* __restrict__ w,
                                   const float* __restrict__ bias, float* __restrict__ state,
                                   const int* __restrict__ cu_q, const int* __restrict__ state_slots,
                                   TO* __restrict__ out, int out_stride, int C, int taps, int residual,
-                                  const float* __restrict__ in_bias) {
+                                  const float* __restrict__ in_bias, int silu, StepSizes ss) {
     pdl_trigger();
     pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     const int e = blockIdx.y;
-    if (c >= C) return;
+    if (c >= C + ss.H) return;
     const int t0 = cu_q[e], q_len = cu_q[e + 1] - t0;
     const int i0 = blockIdx.z * CONV_CHUNK;
     if (i0 >= q_len) return;
+    if (c >= C) {
+        const int h = c - C;
+        const float a = expf(ss.a_log[h]), b = ss.bias[h];
+        for (int i = i0; i < min(q_len, i0 + CONV_CHUNK); ++i) {
+            const float v = to_f32<TI>(x[(size_t)(t0 + i) * x_stride + c]) + b;
+            const float dt = v > 20.f ? v + log1pf(expf(-v)) : log1pf(expf(v));
+            ss.dt[(size_t)(t0 + i) * ss.H + h] = dt;
+            ss.decay[(size_t)(t0 + i) * ss.H + h] = expf(-a * dt);
+        }
+        return;
+    }
     const int back = taps - 1;
     float* st = state + ((size_t)state_slots[e] * back) * C + c;
     float wt[CONV_MAX_TAPS], win[CONV_MAX_TAPS - 1], old[CONV_MAX_TAPS - 1];
@@ -225,6 +246,7 @@ __global__ void short_conv_kernel(const TI* __restrict__ x, int x_stride, const 
 #pragma unroll
         for (int k = 0; k < CONV_MAX_TAPS - 1; ++k)
             if (k < back) y = fmaf(wt[back - 1 - k], win[k], y);
+        if (silu) y = y / (1.0f + expf(-y));
         out[(size_t)(t0 + i) * out_stride + c] = from_f32<TO>(y);
 #pragma unroll
         for (int k = CONV_MAX_TAPS - 2; k > 0; --k) win[k] = win[k - 1];
@@ -517,17 +539,20 @@ RI_API int ri_rms_sandwich(const float* h_in, int in_stride, const void* delta, 
 RI_API int ri_short_conv_max_taps() { return CONV_MAX_TAPS; }
 
 // x rows of x_stride (RI_F32 or RI_BF16), w fp32 [C][taps], bias and in_bias fp32 [C] or null, state fp32 [slots][taps-1][C],
-// out rows of out_stride of out_dtype.  max_q_len: an upper bound of the entries' token counts.
+// out rows of out_stride of out_dtype.  max_q_len: an upper bound of the entries' token counts.  silu: the activation after
+// the bias.  dt_heads > 0: the columns C .. C + dt_heads - 1 of x become step sizes (see StepSizes).
 RI_API int ri_short_conv(const void* x, int x_dtype, int x_stride, const float* w, const float* bias, float* state,
                          const int* cu_q, const int* state_slots, void* out, int out_dtype, int out_stride,
-                         int n_entries, int max_q_len, int C, int taps, int residual, const float* in_bias,
-                         void* stream) {
+                         int n_entries, int max_q_len, int C, int taps, int residual, const float* in_bias, int silu,
+                         const float* dt_bias, const float* a_log, float* dt, float* decay, int dt_heads, void* stream) {
     if (n_entries <= 0 || max_q_len <= 0) return 0;
-    if (taps < 1 || taps > CONV_MAX_TAPS) return (int)cudaErrorInvalidValue;
+    if (taps < 1 || taps > CONV_MAX_TAPS || dt_heads < 0 || (dt_heads > 0 && (!dt_bias || !a_log || !dt || !decay)))
+        return (int)cudaErrorInvalidValue;
+    const StepSizes sizes{dt_bias, a_log, dt, decay, dt_heads};
     cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid((C + 127) / 128, n_entries, (max_q_len + CONV_CHUNK - 1) / CONV_CHUNK);
+    const dim3 grid((C + dt_heads + 127) / 128, n_entries, (max_q_len + CONV_CHUNK - 1) / CONV_CHUNK);
 #define RI_SC(TI, TO) RI_CHECKED(ri_launch(short_conv_kernel<TI, TO>, grid, dim3(128), 0, s, (const TI*)x, x_stride, w, bias, \
-        state, cu_q, state_slots, (TO*)out, out_stride, C, taps, residual, in_bias))
+        state, cu_q, state_slots, (TO*)out, out_stride, C, taps, residual, in_bias, silu, sizes))
     if (x_dtype == RI_BF16) { if (out_dtype == RI_BF16) RI_SC(bf16, bf16); else RI_SC(bf16, float); }
     else { if (out_dtype == RI_BF16) RI_SC(float, bf16); else RI_SC(float, float); }
 #undef RI_SC

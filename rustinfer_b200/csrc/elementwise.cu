@@ -349,9 +349,9 @@ RI_API int ri_rope_scatter(void* qkv, int act_dtype, int row_stride, const int* 
 }
 
 // ------------------------------------------------------------------ SiLU(gate) * up
-// gu row: [gate (I) | up (I)]; out[t, j] = gate / (1 + e^-gate) * up.
+// gu row: [gate (I) | up (I)]; out[t, j] = gate / (1 + e^-gate) * up, or with `gelu` the tanh form of gelu(gate) * up.
 template <typename TA>
-__global__ void silu_mul_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int inter) {
+__global__ void silu_mul_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int inter, int gelu) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.y;
@@ -359,7 +359,8 @@ __global__ void silu_mul_kernel(const TA* __restrict__ gu, TA* __restrict__ out,
     if (j >= inter) return;
     const TA* row = gu + (size_t)t * 2 * inter;
     const float g = to_f32<TA>(row[j]), u = to_f32<TA>(row[inter + j]);
-    out[(size_t)t * inter + j] = from_f32<TA>(g / (1.0f + expf(-g)) * u);
+    const float a = gelu ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.0f + expf(-g));
+    out[(size_t)t * inter + j] = from_f32<TA>(a * u);
 }
 
 // bf16, width a multiple of 8: 16 bytes of gate and of up per thread
@@ -381,10 +382,10 @@ __global__ void silu_mul_bf16x8_kernel(const bf16* __restrict__ gu, bf16* __rest
     }
 }
 
-RI_API int ri_silu_mul(const void* gu, void* out, int act_dtype, int tokens, int inter, void* stream) {
+RI_API int ri_silu_mul(const void* gu, void* out, int act_dtype, int tokens, int inter, int gelu, void* stream) {
     if (tokens <= 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
-    if (act_dtype == RI_BF16 && inter % 8 == 0 && aligned16(gu) && aligned16(out)) {
+    if (!gelu && act_dtype == RI_BF16 && inter % 8 == 0 && aligned16(gu) && aligned16(out)) {
         const size_t n_vec = (size_t)tokens * (inter / 8);
         size_t blocks = (n_vec + 255) / 256;
         if (blocks > (size_t)ri_device_sms() * 16) blocks = (size_t)ri_device_sms() * 16;
@@ -392,8 +393,8 @@ RI_API int ri_silu_mul(const void* gu, void* out, int act_dtype, int tokens, int
         return ri_launch_status();
     }
     dim3 grid((inter + 255) / 256, tokens);
-    if (act_dtype == RI_BF16) RI_CHECKED(ri_launch(silu_mul_kernel<bf16>, dim3(grid), dim3(256), 0, s, (const bf16*)gu, (bf16*)out, inter));
-    else RI_CHECKED(ri_launch(silu_mul_kernel<float>, dim3(grid), dim3(256), 0, s, (const float*)gu, (float*)out, inter));
+    if (act_dtype == RI_BF16) RI_CHECKED(ri_launch(silu_mul_kernel<bf16>, dim3(grid), dim3(256), 0, s, (const bf16*)gu, (bf16*)out, inter, gelu));
+    else RI_CHECKED(ri_launch(silu_mul_kernel<float>, dim3(grid), dim3(256), 0, s, (const float*)gu, (float*)out, inter, gelu));
     return ri_launch_status();
 }
 

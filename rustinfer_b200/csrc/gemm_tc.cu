@@ -36,7 +36,8 @@ constexpr int BM = 128;                 // rows of the A operand per tile (MMA M
 constexpr int BK = 64;                  // 64 bf16 = one 128-byte swizzle row
 constexpr int THREADS = 192;
 
-enum Epilogue { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU = 2, EPI_RESIDUAL = 3, EPI_ROPE = 4, EPI_RELU2 = 5 };
+enum Epilogue { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU = 2, EPI_RESIDUAL = 3, EPI_ROPE = 4, EPI_RELU2 = 5, EPI_GELU = 6 };
+// EPI_GELU: EPI_SILU with the pair gelu_tanh(gate) * up (the kernels see EPI_SILU and glu_gelu)
 // EPI_RELU2: max(x, 0)^2 of the fp32 sum, stored bf16 (the activation of a feed-forward without a gate)
 __device__ __forceinline__ float relu2(float x) { return x > 0.f ? x * x : 0.f; }
 enum ErrorCode { ERR_PRODUCER_WAIT = 1, ERR_MMA_WAIT = 2, ERR_EPILOGUE_WAIT = 3, ERR_DRAIN_WAIT = 4 };
@@ -102,6 +103,7 @@ struct Params {
     // EPI_SILU with glu_limit > 0: the pair (gate g, up u) becomes g' sigmoid(glu_alpha g') (u' + 1) with
     // g' = min(g, glu_limit), u' = clamp(u, -glu_limit, glu_limit) instead of silu(g) u
     float glu_limit = 0.f, glu_alpha = 0.f;
+    int glu_gelu = 0;                    // EPI_SILU: gelu(g) u with gelu(g) = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))
 };
 
 __device__ __forceinline__ float glu_mul(const Params& p, float g, float u) {
@@ -109,6 +111,11 @@ __device__ __forceinline__ float glu_mul(const Params& p, float g, float u) {
         g = fminf(g, p.glu_limit);
         u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
         return __fdividef(g, 1.0f + __expf(-p.glu_alpha * g)) * (u + 1.0f);
+    }
+    if (p.glu_gelu) {
+        // 0.5 (1 + tanh(y)) = 1 / (1 + e^(-2y))
+        const float y = 0.7978845608028654f * (g + 0.044715f * g * g * g);
+        return __fdividef(g, 1.0f + __expf(-2.0f * y)) * u;
     }
     return silu_mul(g, u);
 }
@@ -968,7 +975,8 @@ RI_API long long ri_gemm_tc_workspace_floats(int M, int N, int splits, int swap,
 
 // X [M][K] bf16 (row pitch K), W [N][K] bf16; out per `epilogue`:
 //   0 bf16 [M][ld_out], 1 fp32 [M][ld_out], 2 bf16 [M][ld_out] = silu(gate)*up with W's rows
-//   alternating gate_j, up_j (N = 2 * features of out), 3 fp32 [M][ld_out] += result.
+//   alternating gate_j, up_j (N = 2 * features of out), 3 fp32 [M][ld_out] += result, 5 bf16 max(x, 0)^2,
+//   6 as 2 with gelu_tanh(gate) * up.
 // swap: 1 puts the weight on the 128-row side of the MMA (few tokens), 0 the activations.
 // bn: rows of the other operand per tile (16, 32, 64, 128 or 256).  counters: one int per
 // tile, zero before the first call (the kernel leaves them zero).  error: one int that a
@@ -995,6 +1003,7 @@ int gemm_tc_impl(const void* X, const void* W, int M, int N, int K, void* out, i
     const void* A = swap ? W : X;
     const void* B = swap ? X : W;
     Params p;
+    if (epilogue == EPI_GELU) { p.glu_gelu = 1; epilogue = EPI_SILU; }
     p.pair_bn = 0;
     p.sk_tiles = p.sk_pairs = p.sk_q = p.sk_extra = 0; p.sk_acc = nullptr;
     p.rope_positions = nullptr; p.rope_cos = p.rope_sin = nullptr; p.rope_slot = nullptr; p.rope_cache = nullptr;

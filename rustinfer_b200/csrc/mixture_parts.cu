@@ -7,12 +7,13 @@
 //            counts[e] += 1 (or from given logits z [T][E])
 //   sort     ids, counts -> offsets [E+1], order [T*top] (pairs in expert order, stable), place [T*top]
 //   products rows of an expert times that expert's matrix (fp32 sums in a fixed order of k)
-//   combine  y[t] = sum_j weight[t][j] * Y[place[t*top + j]] (+ shared[t]); counts put back to zero
+//   combine  y[t] = sum_j weight[t][j] * Y[place[t*top + j]] (+ gate[t] * shared[t]); counts put back to zero
 #include "common.cuh"
 
 namespace {
 
 // ------------------------------------------------------------------------------- router
+// (score 2: s = softmax(z) over all experts; group_max: a group's score is its largest c; gate: see below.)
 // One CTA a token.  Logit z_e = sum_i W[e][i] x[i] in fp32 (a lane every 32nd term, then a butterfly over the
 // lanes: the same order whatever else is in the batch) unless the logits are given; then one warp chooses.  score s = sigmoid(z);
 // choice c = s + correction.  With groups: the experts form
@@ -35,20 +36,23 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS)
 moe_route_kernel(const float* __restrict__ z, const TX* __restrict__ x, const float* __restrict__ router,
                  int d, const float* __restrict__ correction, int T, int E,
                  int top, int n_groups, int keep, int renorm, int* __restrict__ ids,
-                 float* __restrict__ weights, int* __restrict__ counts, int score) {
+                 float* __restrict__ weights, int* __restrict__ counts, int score, int group_max, float renorm_eps,
+                 float* __restrict__ gate) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
-    float* s = sm;                                         // [E] scores
-    float* c = s + E;                                      // [E] choice scores
+    // gate (with x): the router's matrix has one row more, whose product's sigmoid goes to gate[t]
+    const int rows = E + (gate && x ? 1 : 0);
+    float* s = sm;                                         // [rows] scores
+    float* c = s + rows;                                   // [E] choice scores
     float* gs = c + E;                                     // [n_groups] group scores
     if (x) {
         // the logits: the warps share the experts, eight at a time; a lane takes every 32nd term of all eight
         // sums (x is read once for them), then the lanes' parts meet in a butterfly
         const TX* xr = x + (size_t)t * d;
-        for (int e0 = warp * ROUTE_CHUNK; e0 < E; e0 += ROUTE_WARPS * ROUTE_CHUNK) {
+        for (int e0 = warp * ROUTE_CHUNK; e0 < rows; e0 += ROUTE_WARPS * ROUTE_CHUNK) {
             float acc[ROUTE_CHUNK];
 #pragma unroll
             for (int j = 0; j < ROUTE_CHUNK; ++j) acc[j] = 0.f;
@@ -57,21 +61,29 @@ moe_route_kernel(const float* __restrict__ z, const TX* __restrict__ x, const fl
                 const float xv = to_f32<TX>(xr[i]);
 #pragma unroll
                 for (int j = 0; j < ROUTE_CHUNK; ++j)
-                    if (e0 + j < E) acc[j] = fmaf(xv, router[(size_t)(e0 + j) * d + i], acc[j]);
+                    if (e0 + j < rows) acc[j] = fmaf(xv, router[(size_t)(e0 + j) * d + i], acc[j]);
             }
 #pragma unroll
             for (int j = 0; j < ROUTE_CHUNK; ++j) {
                 const float dot = warp_sum(acc[j]);
-                if (lane == 0 && e0 + j < E) s[e0 + j] = dot;
+                if (lane == 0 && e0 + j < rows) s[e0 + j] = dot;
             }
         }
         __syncthreads();
     }
     if (warp != 0) return;                                 // the choice is one warp's work
+    if (gate && x && lane == 0) gate[t] = 1.0f / (1.0f + expf(-s[E]));
+    float zmx = -INFINITY, zsum = 0.f;                     // of the softmax over all experts
+    if (score == 2) {
+        for (int e = lane; e < E; e += 32) zmx = fmaxf(zmx, x ? s[e] : z[(size_t)t * E + e]);
+        zmx = warp_max(zmx);
+        for (int e = lane; e < E; e += 32) zsum += expf((x ? s[e] : z[(size_t)t * E + e]) - zmx);
+        zsum = warp_sum(zsum);
+    }
     for (int e = lane; e < E; e += 32) {
         // score 0: the sigmoid of the logit; 1: the logit itself, the chosen ones' weights their softmax
         const float zl = x ? s[e] : z[(size_t)t * E + e];
-        const float sc = score == 1 ? zl : 1.0f / (1.0f + expf(-zl));
+        const float sc = score == 1 ? zl : score == 2 ? expf(zl - zmx) / zsum : 1.0f / (1.0f + expf(-zl));
         s[e] = sc;
         c[e] = sc + (correction ? correction[e] : 0.f);
     }
@@ -84,7 +96,7 @@ moe_route_kernel(const float* __restrict__ z, const TX* __restrict__ x, const fl
                 const float v = c[g * per + i];
                 if (v > a) { b = a; a = v; } else if (v > b) b = v;
             }
-            gs[g] = per > 1 ? a + b : a;
+            gs[g] = per > 1 && !group_max ? a + b : a;
         }
         __syncwarp();
         // the `keep` best groups get +inf as a mark, one by one
@@ -130,7 +142,7 @@ moe_route_kernel(const float* __restrict__ z, const TX* __restrict__ x, const fl
     if (score == 1) {
         if (lane < top) weights[(size_t)t * top + lane] = expf(weights[(size_t)t * top + lane] - zmax) / wsum;
     } else if (renorm && lane < top) {
-        weights[(size_t)t * top + lane] /= wsum;
+        weights[(size_t)t * top + lane] /= wsum + renorm_eps;
     }
 }
 
@@ -455,11 +467,11 @@ __global__ void moe_gather_kernel(const bf16* __restrict__ x, const int* __restr
 }
 
 // ------------------------------------------------------------------------------ combine
-// out[t][c] = sum_j weights[t][j] * Y[place[t*top + j]][c] (+ shared[t][c]), j = 0, 1, .. in that order.
+// out[t][c] = sum_j weights[t][j] * Y[place[t*top + j]][c] (+ gate[t] shared[t][c]; gate null: 1), j = 0, 1, .. in order.
 template <typename TS, typename TO>
 __global__ void moe_combine_kernel(const float* __restrict__ Y, const int* __restrict__ place,
                                    const float* __restrict__ weights, const TS* __restrict__ shared, TO* __restrict__ out,
-                                   int top, int d, int* __restrict__ counts, int E) {
+                                   int top, int d, int* __restrict__ counts, int E, const float* __restrict__ gate) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -469,32 +481,35 @@ __global__ void moe_combine_kernel(const float* __restrict__ Y, const int* __res
         float acc = 0.f;
         for (int j = 0; j < top; ++j)
             acc = fmaf(weights[(size_t)t * top + j], Y[(size_t)place[(size_t)t * top + j] * d + c], acc);
-        if (shared) acc += to_f32<TS>(shared[(size_t)t * d + c]);
+        if (shared) acc = fmaf(gate ? gate[t] : 1.f, to_f32<TS>(shared[(size_t)t * d + c]), acc);
         out[(size_t)t * d + c] = from_f32<TO>(acc);
     }
 }
 
 }  // namespace
 
-// Either z (fp32 [T][E]) or x ([T][d] of x_dtype) with router (fp32 [E][d]) is given.
+// Either z (fp32 [T][E]) or x ([T][d] of x_dtype) with router (fp32 [E][d], [E + 1][d] with gate) is given.
 RI_API int ri_moe_route(const float* z, const void* x, int x_dtype, const float* router, int d, const float* correction,
                         int T, int E, int top, int n_groups, int keep,
-                        int renorm, int* ids, float* weights, int* counts, int score, void* stream) {
+                        int renorm, int* ids, float* weights, int* counts, int score, int group_max, float renorm_eps,
+                        float* gate, void* stream) {
     if (T <= 0) return 0;
-    if (score != 0 && score != 1) return (int)cudaErrorInvalidValue;
+    if (score < 0 || score > 2 || (gate && !x)) return (int)cudaErrorInvalidValue;
     if (E <= 0 || top <= 0 || top > E || top > 32 || (n_groups > 0 && (E % n_groups || keep <= 0 || keep > n_groups)))
         return (int)cudaErrorInvalidValue;
     const int warps = ROUTE_WARPS;
-    const size_t smem = (size_t)(2 * E + (n_groups > 0 ? n_groups : 0)) * sizeof(float);
+    const size_t smem = (size_t)(2 * E + 1 + (n_groups > 0 ? n_groups : 0)) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     if ((z == nullptr) == (x == nullptr) || (x && !router)) return (int)cudaErrorInvalidValue;
     const dim3 grid(T);
     if (x && x_dtype == RI_BF16)
         RI_CHECKED(ri_launch(moe_route_kernel<bf16>, grid, dim3(32 * warps), smem, (cudaStream_t)stream, z, (const bf16*)x, router, d,
-                             correction, T, E, top, n_groups > 0 ? n_groups : 0, keep, renorm, ids, weights, counts, score));
+                             correction, T, E, top, n_groups > 0 ? n_groups : 0, keep, renorm, ids, weights, counts, score,
+                             group_max, renorm_eps, gate));
     else
         RI_CHECKED(ri_launch(moe_route_kernel<float>, grid, dim3(32 * warps), smem, (cudaStream_t)stream, z, (const float*)x, router, d,
-                             correction, T, E, top, n_groups > 0 ? n_groups : 0, keep, renorm, ids, weights, counts, score));
+                             correction, T, E, top, n_groups > 0 ? n_groups : 0, keep, renorm, ids, weights, counts, score,
+                             group_max, renorm_eps, gate));
     return ri_launch_status();
 }
 
@@ -580,11 +595,11 @@ RI_API int ri_moe_gather(const void* x, const int* order, int top, void* out, in
 }
 
 RI_API int ri_moe_combine(const float* Y, const int* place, const float* weights, const void* shared, int shared_dtype,
-                          void* out, int out_dtype, int T, int top, int d, int* counts, int E, void* stream) {
+                          void* out, int out_dtype, int T, int top, int d, int* counts, int E, const float* gate, void* stream) {
     if (T <= 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
 #define RI_MC(TS, TO) RI_CHECKED(ri_launch(moe_combine_kernel<TS, TO>, dim3(T), dim3(256), 0, s, Y, place, weights, \
-        (const TS*)shared, (TO*)out, top, d, counts, E))
+        (const TS*)shared, (TO*)out, top, d, counts, E, gate))
     if (shared_dtype == RI_BF16 && out_dtype == RI_BF16) RI_MC(bf16, bf16);
     else if (shared_dtype == RI_BF16) RI_MC(bf16, float);
     else if (out_dtype == RI_BF16) RI_MC(float, bf16);

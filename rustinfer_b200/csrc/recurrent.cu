@@ -2,10 +2,13 @@
 // kept in fp32 (compiled for one key size RI_KDIM; any value size):
 //
 //   gated      S_t = diag(alpha_t) S_{t-1} + k_t v_t^T                          o_t = S_t^T q_t
+//   head       S_t = a_t S_{t-1} + k_t (g_t v_t)^T, a and g one number a head   o_t = S_t^T q_t
 //   delta      S_t = diag(w_t) S_{t-1} - (a_t * u_t)(u_t^T S_{t-1}) + k_t v_t^T   o_t = S_t^T r_t
 //
 // The decays alpha and w, the unit keys u and the products a * u arrive as fp32 vectors per token
-// (made from the projections by kernels that run over all tokens at once, sequence_parts.cu).
+// (made from the projections by kernels that run over all tokens at once, sequence_parts.cu).  The "head" form serves
+// decays that are one number a head, fixed (retention) or per token (a state-space recurrence with step sizes g);
+// several heads may share keys and queries, and single tokens may have theirs rotated on the way in.
 //
 // The columns of S do not mix, so a CTA owns a tile of value channels of one head of one batch
 // entry and walks the entry's tokens in order, whatever their number: a prompt, a portion of
@@ -571,6 +574,188 @@ delta_scan_kernel(const TA* __restrict__ r, int r_stride, const TA* __restrict__
     if (!loader) store_state(S, sp, ok);
 }
 
+// ------------------------------------------------------------- one decay a head
+// As the gated walk, but a token's decay is one number a head, a_t, its values may be multiplied by another, g_t, and
+// heads share keys and queries in groups of `share` (head h reads key head h / share):
+//   S <- a S + k (g v);   o += S q
+struct HeadHalf {
+    float *q, *k, *v, *a;
+    __device__ HeadHalf(float* base) : q(base), k(base + TC * ROWLEN), v(base + 2 * TC * ROWLEN), a(v + TC * COLS) {}
+};
+constexpr int HEAD_HALF = 2 * TC * ROWLEN + TC * COLS + TC;
+
+__device__ __forceinline__ void head_rows(float* S, float a, const float4& k, const float4& q, float vj, float& o0, float& o1) {
+    S[0] = fmaf(a, S[0], k.x * vj);
+    S[1] = fmaf(a, S[1], k.y * vj);
+    S[2] = fmaf(a, S[2], k.z * vj);
+    S[3] = fmaf(a, S[3], k.w * vj);
+    o0 = fmaf(S[0], q.x, o0);
+    o1 = fmaf(S[1], q.y, o1);
+    o0 = fmaf(S[2], q.z, o0);
+    o1 = fmaf(S[3], q.w, o1);
+}
+
+__device__ __forceinline__ void head_token(float (&S)[C][NR], const HeadHalf& b, int tok, int rg, int cg, float (&part)[C]) {
+    const float4* k4 = reinterpret_cast<const float4*>(b.k + tok * ROWLEN + rg * NRP);
+    const float4* q4 = reinterpret_cast<const float4*>(b.q + tok * ROWLEN + rg * NRP);
+    const float a = b.a[tok];
+    float vj[C], o0[C], o1[C];
+#pragma unroll
+    for (int j = 0; j < C; ++j) {
+        vj[j] = b.v[tok * COLS + cg * C + j];
+        o0[j] = o1[j] = 0.f;
+    }
+#pragma unroll
+    for (int m = 0; m < NR / 4; ++m) {
+        const float4 kk = k4[m], qq = q4[m];
+#pragma unroll
+        for (int j = 0; j < C; ++j) head_rows(&S[j][4 * m], a, kk, qq, vj[j], o0[j], o1[j]);
+    }
+#pragma unroll
+    for (int j = 0; j < C; ++j) part[j] = o0[j] + o1[j];
+}
+
+// q, k: [T, >= H/share*DK] with row strides; v: [T, >= H*dv]; decay: fp32, decay[t * a_stride + h] (a_stride 0: the same for
+// every token); gain: fp32 [T][g_stride], or null (1); out: fp32 [T, H*dv]; state: [slots][H][dv][DKP] fp32.
+template <typename TA>
+__global__ void __launch_bounds__(THREADS, DK <= 128 ? 2 : 1)
+head_scan_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ k, int k_stride, const TA* __restrict__ v,
+                 int v_stride, const float* __restrict__ decay, int a_stride, const float* __restrict__ gain, int g_stride,
+                 float q_scale, float* __restrict__ out, float* __restrict__ state, const int* __restrict__ cu_q,
+                 const int* __restrict__ state_slots, int H, int dv, int share, int vec) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float smem[];
+    const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS;
+    const int kh = h / share;
+    const int tid = threadIdx.x;
+    const bool loader = tid >= WORKERS;
+    const int lt = tid - WORKERS;
+    const int cg = tid / R, rg = tid % R;
+    const int t_begin = cu_q[b], t_end = cu_q[b + 1];
+    const int rounds = (t_end - t_begin + TC - 1) / TC;
+    if (DKP != DK) {                                         // rows beyond DK stay zero
+        for (int e = tid; e < 2 * HEAD_HALF; e += THREADS) smem[e] = 0.f;
+        __syncthreads();
+    }
+
+    auto stage = [&](int round) {
+        const HeadHalf hb(smem + (round & 1) * HEAD_HALF);
+        const int t0 = t_begin + round * TC, nt = min(TC, t_end - t0);
+        float vv[PERV];
+        load_values(vv, v, v_stride, t0, nt, h, dv, c0, lt);
+        if (gain) {
+#pragma unroll
+            for (int j = 0; j < PERV; ++j) {
+                const int tok = min(lt + j * WORKERS, nt * COLS - 1) / COLS;
+                vv[j] *= gain[(size_t)(t0 + tok) * g_stride + h];
+            }
+        }
+        const float av = decay[(size_t)(t0 + min(lt, nt - 1)) * a_stride + h];
+        if (vec) {                                           // loads unconditional, as in the gated kernel
+            float4 qv[PER4], kv[PER4];
+#pragma unroll
+            for (int j = 0; j < PER4; ++j) {
+                const int e = min(lt + j * WORKERS, nt * (DK / 4) - 1);
+                const int tok = e / (DK / 4), i = (e - tok * (DK / 4)) * 4;
+                const size_t t = (size_t)(t0 + tok), c = (size_t)kh * DK + i;
+                qv[j] = ld4(q + t * q_stride + c);
+                kv[j] = ld4(k + t * k_stride + c);
+            }
+#pragma unroll
+            for (int j = 0; j < PER4; ++j) {
+                const int e = lt + j * WORKERS;
+                if (e < nt * (DK / 4)) {
+                    const int tok = e / (DK / 4), i = (e - tok * (DK / 4)) * 4;
+                    const int at = tok * ROWLEN + row_at(i);
+                    *reinterpret_cast<float4*>(hb.q + at) = scaled(qv[j], q_scale);
+                    *reinterpret_cast<float4*>(hb.k + at) = kv[j];
+                }
+            }
+        } else {
+            float qv[PER], kv[PER];
+#pragma unroll
+            for (int j = 0; j < PER; ++j) {
+                const int e = min(lt + j * WORKERS, nt * DK - 1);
+                const int tok = e / DK, i = e - tok * DK;
+                const size_t t = (size_t)(t0 + tok), c = (size_t)kh * DK + i;
+                qv[j] = ld(q, t * q_stride + c);
+                kv[j] = ld(k, t * k_stride + c);
+            }
+#pragma unroll
+            for (int j = 0; j < PER; ++j) {
+                const int e = lt + j * WORKERS;
+                if (e < nt * DK) {
+                    const int tok = e / DK, i = e - tok * DK;
+                    const int at = tok * ROWLEN + row_at(i);
+                    hb.q[at] = qv[j] * q_scale;
+                    hb.k[at] = kv[j];
+                }
+            }
+        }
+        store_values(hb.v, vv, nt, dv, c0, lt);
+        if (lt < nt) hb.a[lt] = av;
+    };
+
+    bool ok[C];
+#pragma unroll
+    for (int j = 0; j < C; ++j) ok[j] = !loader && c0 + cg * C + j < dv;
+    float* sp = nullptr;
+    float S[C][NR];
+    if (loader) {
+        if (rounds > 0) stage(0);
+    } else {
+        sp = state + ((((size_t)state_slots[b] * H + h) * dv + c0 + cg * C) * DKP + rg * NR);
+        load_state(S, sp, ok);
+    }
+    __syncthreads();
+    for (int round = 0; round < rounds; ++round) {
+        if (loader) {
+            if (round + 1 < rounds) stage(round + 1);
+        } else {
+            const HeadHalf hb(smem + (round & 1) * HEAD_HALF);
+            const int t0 = t_begin + round * TC, nt = min(TC, t_end - t0);
+            float* op = out + ((size_t)t0 * H + h) * dv + c0 + cg * C;
+            if (nt == TC) {
+#pragma unroll
+                for (int tb = 0; tb < TC; tb += TB) {        // the outputs' sums in batches, as in the gated kernel
+                    GroupSums<TB * C> sums;                  // value i * C + j: token tb + i, column j
+#pragma unroll
+                    for (int i = 0; i < TB; ++i) {
+                        float part[C];
+                        head_token(S, hb, tb + i, rg, cg, part);
+#pragma unroll
+                        for (int j = 0; j < C; ++j) sums.x[i * C + j] = part[j];
+                    }
+                    sums.run(rg);
+                    if (sums.owner) {
+#pragma unroll
+                        for (int n = 0; n < TB * C; ++n) {
+                            if (n < sums.count) {
+                                const int idx = sums.first + n, i = idx / C, j = idx - i * C;
+                                if (c0 + cg * C + j < dv) op[(size_t)(tb + i) * H * dv + j] = sums.x[n];
+                            }
+                        }
+                    }
+                }
+            } else {
+#pragma unroll 1
+                for (int tok = 0; tok < nt; ++tok) {
+                    float part[C];
+                    head_token(S, hb, tok, rg, cg, part);
+#pragma unroll
+                    for (int j = 0; j < C; ++j) {
+                        const float o = group_sum(part[j]);
+                        if (rg == 0 && ok[j]) op[(size_t)tok * H * dv + j] = o;
+                    }
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (!loader) store_state(S, sp, ok);
+}
+
 // ------------------------------------------------------------- entries of a single token
 // A step in which every entry brings one token (decoding): no rounds and no staging.  A CTA of
 // WORKERS threads owns COLS value channels of one head of one entry; a lane reads its rows of the
@@ -665,6 +850,78 @@ delta_step_kernel(const TA* __restrict__ r, int r_stride, const TA* __restrict__
     store_state(S, sp, ok);
 }
 
+// Rotation of the keys and queries a step of single tokens reads: the first `rot` channels of a head turn by the angles
+// of the token's position (cos / sin [positions][rot / 2]); cos null: none.  Pairs (i, i + rot/2), or (2i, 2i+1).
+struct StepRotation {
+    const int* positions;
+    const float *cos_t, *sin_t;
+    int rot, interleaved;
+};
+template <typename TA>
+__device__ __forceinline__ void rotated_rows_of(float4 (&x)[NR / 4], const TA* p, int rg, float scale, const StepRotation& ro, int pos) {
+    if (!ro.cos_t) { rows_of(x, p, rg, scale); return; }
+    const int half = ro.rot >> 1;
+#pragma unroll
+    for (int m = 0; m < NR / 4; ++m) {
+        float e[4];
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+            const int i = rg * NR + 4 * m + n;
+            e[n] = 0.f;
+            if (i < DK) {
+                const float own = to_f32<TA>(p[i]);
+                if (i < ro.rot) {
+                    const int pair = ro.interleaved ? i >> 1 : i < half ? i : i - half;
+                    const bool first = ro.interleaved ? (i & 1) == 0 : i < half;
+                    const float other = to_f32<TA>(p[ro.interleaved ? i ^ 1 : first ? i + half : i - half]);
+                    const float c = ro.cos_t[(size_t)pos * half + pair], s = ro.sin_t[(size_t)pos * half + pair];
+                    e[n] = (first ? own * c - other * s : own * c + other * s) * scale;
+                } else {
+                    e[n] = own * scale;
+                }
+            }
+        }
+        x[m] = make_float4(e[0], e[1], e[2], e[3]);
+    }
+}
+
+template <typename TA>
+__global__ void __launch_bounds__(WORKERS)
+head_step_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ k, int k_stride, const TA* __restrict__ v,
+                 int v_stride, const float* __restrict__ decay, int a_stride, const float* __restrict__ gain, int g_stride,
+                 float q_scale, float* __restrict__ out, float* __restrict__ state, const int* __restrict__ cu_q,
+                 const int* __restrict__ state_slots, int H, int dv, int share, StepRotation ro) {
+    pdl_trigger();
+    pdl_wait();
+    const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS;
+    const int kh = h / share;
+    const int cg = threadIdx.x / R, rg = threadIdx.x % R;
+    const int t = cu_q[b];
+    if (cu_q[b + 1] - t != 1) return;                        // the host sends only steps of single tokens here
+    bool ok[C];
+#pragma unroll
+    for (int j = 0; j < C; ++j) ok[j] = c0 + cg * C + j < dv;
+    float* sp = state + ((((size_t)state_slots[b] * H + h) * dv + c0 + cg * C) * DKP + rg * NR);
+    float S[C][NR];
+    load_state(S, sp, ok);
+    const float a = decay[(size_t)t * a_stride + h], g = gain ? gain[(size_t)t * g_stride + h] : 1.f;
+    const int pos = ro.cos_t ? ro.positions[t] : 0;
+    float4 kk[NR / 4], qq[NR / 4];
+    rotated_rows_of(kk, k + (size_t)t * k_stride + (size_t)kh * DK, rg, 1.f, ro, pos);
+    rotated_rows_of(qq, q + (size_t)t * q_stride + (size_t)kh * DK, rg, q_scale, ro, pos);
+#pragma unroll
+    for (int j = 0; j < C; ++j) {
+        float vj = ok[j] ? to_f32<TA>(v[(size_t)t * v_stride + (size_t)h * dv + c0 + cg * C + j]) : 0.f;
+        if (gain) vj *= g;
+        float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+        for (int m = 0; m < NR / 4; ++m) head_rows(&S[j][4 * m], a, kk[m], qq[m], vj, o0, o1);
+        const float o = group_sum(o0 + o1);
+        if (rg == 0 && ok[j]) out[((size_t)t * H + h) * dv + c0 + cg * C + j] = o;
+    }
+    store_state(S, sp, ok);
+}
+
 inline bool aligned4(const void* p, int esize) { return (reinterpret_cast<uintptr_t>(p) % (4 * (size_t)esize)) == 0; }
 
 template <typename Kernel>
@@ -731,6 +988,39 @@ RI_API int ri_delta_scan(const void* r, int r_stride, const void* k, int k_strid
     if (act_dtype == RI_BF16) RI_DS(bf16);
     else RI_DS(float);
 #undef RI_DS
+    return ri_launch_status();
+}
+
+// The head form: see head_scan_kernel.  share: heads that read one key head.  cos_t / sin_t with positions (with `single`
+// only; else null): keys and queries are rotated on the way in (see StepRotation).
+RI_API int ri_head_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
+                        const float* decay, int a_stride, const float* gain, int g_stride, int act_dtype, float q_scale,
+                        float* out, float* state, const int* cu_q, const int* state_slots, int entries, int H, int dv,
+                        int share, const int* positions, const float* cos_t, const float* sin_t, int rot, int interleaved,
+                        int single, void* stream) {
+    if (entries <= 0) return 0;
+    if (share <= 0 || H % share || (cos_t && (!single || !positions || !sin_t || rot < 2 || rot > DK || (rot & 1))))
+        return (int)cudaErrorInvalidValue;
+    cudaStream_t s = (cudaStream_t)stream;
+    const dim3 grid((dv + COLS - 1) / COLS, H, entries);
+    const size_t smem = 2 * (size_t)HEAD_HALF * sizeof(float);
+    const int esize = act_dtype == RI_BF16 ? 2 : 4;
+    const int vec = DK % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && aligned4(q, esize) && aligned4(k, esize);
+    const StepRotation ro{positions, cos_t, sin_t, rot, interleaved};
+#define RI_HS(TA) do { \
+    if (single) { \
+        RI_CHECKED(ri_launch(head_step_kernel<TA>, grid, dim3(WORKERS), 0, s, (const TA*)q, q_stride, (const TA*)k, k_stride, \
+            (const TA*)v, v_stride, decay, a_stride, gain, g_stride, q_scale, out, state, cu_q, state_slots, H, dv, share, ro)); \
+        break; \
+    } \
+    static bool allowed = false; \
+    if (!allowed) { RI_CHECKED(allow_shared(head_scan_kernel<TA>, smem)); allowed = true; } \
+    RI_CHECKED(ri_launch(head_scan_kernel<TA>, grid, dim3(THREADS), smem, s, (const TA*)q, q_stride, (const TA*)k, k_stride, \
+        (const TA*)v, v_stride, decay, a_stride, gain, g_stride, q_scale, out, state, cu_q, state_slots, H, dv, share, vec)); \
+    } while (0)
+    if (act_dtype == RI_BF16) RI_HS(bf16);
+    else RI_HS(float);
+#undef RI_HS
     return ri_launch_status();
 }
 

@@ -166,13 +166,37 @@ __global__ void hyper_collect_kernel(float* __restrict__ X, int fresh, const TY*
 // `cache` at slot_of_token[t] (page*page_size + offset; < 0 or no cache: not stored).  One CTA a token.
 // Hv: heads of v where they are fewer than the heads of k (several attention maps, each with keys of
 // its own, over one set of values); a page then holds Hkv heads of keys and Hv heads of values.
+// `conv` (w null: none), for a step in which token t is the one token of entry t: every channel first passes a short
+// causal convolution over time, y = sum_j w[c][j] x_(t - taps + 1 + j), whose earlier inputs come from the entry's state
+// slot, which the new input is shifted into (a channel of an entry is one thread's work).
+struct QkvConv {
+    const float* w;              // [channels][taps]
+    float* state;                // [slots][taps - 1][channels], oldest first
+    const int* slots;
+    int taps;
+};
+__device__ __forceinline__ float conv_channel(const QkvConv& cv, int t, int c, int channels, float x) {
+    const int back = cv.taps - 1;
+    const float* wc = cv.w + (size_t)c * cv.taps;
+    float* st = cv.state + (size_t)cv.slots[t] * back * channels + c;
+    float y = wc[back] * x, prev = x;
+    for (int k = back - 1; k >= 0; --k) {
+        const float old = st[(size_t)k * channels];
+        y = fmaf(wc[k], old, y);
+        st[(size_t)k * channels] = prev;
+        prev = old;
+    }
+    return y;
+}
+
 template <typename TI, typename TA, typename TW>
-__global__ void qkv_prepare_kernel(const TI* __restrict__ qkv, int row_stride, const float* __restrict__ bias,
+__global__ void __launch_bounds__(1024) qkv_prepare_kernel(const TI* __restrict__ qkv, int row_stride, const float* __restrict__ bias,
                                    const TW* __restrict__ q_w, const TW* __restrict__ k_w, int norm_mode, float eps,
                                    const int* __restrict__ positions, const float* __restrict__ cos_t,
                                    const float* __restrict__ sin_t, int rot, int interleaved,
                                    const int* __restrict__ slot_of_token, TA* __restrict__ cache,
-                                   TA* __restrict__ q_out, int Hq, int Hkv, int Hv, int dk, int dv, int has_kv, int page_size) {
+                                   TA* __restrict__ q_out, int Hq, int Hkv, int Hv, int dk, int dv, int has_kv, int page_size,
+                                   QkvConv cv) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float sm[];
@@ -186,6 +210,7 @@ __global__ void qkv_prepare_kernel(const TI* __restrict__ qkv, int row_stride, c
     for (int i = tid; i < nq + nk; i += nth) {
         float v = to_f32<TI>(row[i]);
         if (bias) v += bias[i];
+        if (cv.w) v = conv_channel(cv, t, i, nq + nk + (has_kv ? Hv * dv : 0), v);
         sm[i] = v;
         if (i < nq) ssq += v * v; else ssk += v * v;
     }
@@ -228,9 +253,13 @@ __global__ void qkv_prepare_kernel(const TI* __restrict__ qkv, int row_stride, c
         __syncthreads();
     }
     for (int i = tid; i < nq; i += nth) q_out[(size_t)t * nq + i] = from_f32<TA>(qs[i]);
-    if (!has_kv || !cache || !slot_of_token) return;
-    const int slot = slot_of_token[t];
-    if (slot < 0) return;
+    const int slot = has_kv && cache && slot_of_token ? slot_of_token[t] : -1;
+    if (slot < 0) {
+        if (cv.w)                                             // the values' inputs are state all the same
+            for (int i = tid; has_kv && i < Hv * dv; i += nth)
+                conv_channel(cv, t, nq + nk + i, nq + nk + Hv * dv, to_f32<TI>(row[nq + nk + i]) + (bias ? bias[nq + nk + i] : 0.f));
+        return;
+    }
     const size_t page_elems = (size_t)page_size * ((size_t)Hkv * dk + (size_t)Hv * dv);
     TA* page = cache + (size_t)(slot / page_size) * page_elems;
     const int off = slot % page_size;
@@ -244,6 +273,7 @@ __global__ void qkv_prepare_kernel(const TI* __restrict__ qkv, int row_stride, c
         const int g = i / dv, c = i - g * dv;
         float v = to_f32<TI>(row[nq + nk + i]);
         if (bias) v += bias[nq + nk + i];
+        if (cv.w) v = conv_channel(cv, t, nq + nk + i, nq + nk + nv, v);
         vpage[((size_t)g * page_size + off) * dv + c] = from_f32<TA>(v);
     }
 }
@@ -295,13 +325,19 @@ RI_API int ri_hyper_collect(float* X, int fresh, const void* y, int y_dtype, con
     return ri_launch_status();
 }
 
-// in_dtype: of qkv; act_dtype: of q_out and the cache; w_dtype: of the norm weights.  bias is fp32.
+// in_dtype: of qkv; act_dtype: of q_out and the cache; w_dtype: of the norm weights.  bias is fp32.  conv_w (may be null):
+// see QkvConv.
 RI_API int ri_qkv_prepare(const void* qkv, int in_dtype, int row_stride, const float* bias, const void* q_w,
                           const void* k_w, int w_dtype, int norm_mode, float eps, const int* positions,
                           const float* cos_t, const float* sin_t, int rot, int interleaved, const int* slot_of_token,
                           void* cache, void* q_out, int act_dtype, int tokens, int Hq, int Hkv, int dk, int dv,
-                          int has_kv, int page_size, int value_heads, void* stream) {
+                          int has_kv, int page_size, int value_heads, const float* conv_w, float* conv_state,
+                          const int* conv_slots, int conv_taps, void* stream) {
     if (tokens <= 0) return 0;
+    if (conv_w && (!conv_slots || conv_taps < 1 || (conv_taps > 1 && !conv_state))) return (int)cudaErrorInvalidValue;
+    const QkvConv cv{conv_w, conv_state, conv_slots, conv_taps};
+    // with the convolution a step has few tokens and a thread waits for its channel's state: more threads a token
+    const int threads = conv_w ? 1024 : 256;
     const int Hv = value_heads > 0 ? value_heads : Hkv;
     if (rot < 0 || rot > dk || (rot & 1) || (rot > 0 && (!cos_t || !sin_t || !positions))) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
@@ -313,9 +349,9 @@ RI_API int ri_qkv_prepare(const void* qkv, int in_dtype, int row_stride, const f
             cudaError_t e = cudaFuncSetAttribute(qkv_prepare_kernel<TI, TA, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
             if (e != cudaSuccess) return (int)e; \
             configured = true; } \
-        RI_CHECKED(ri_launch(qkv_prepare_kernel<TI, TA, TW>, dim3(tokens), dim3(256), smem, s, (const TI*)qkv, row_stride, bias, \
+        RI_CHECKED(ri_launch(qkv_prepare_kernel<TI, TA, TW>, dim3(tokens), dim3(threads), smem, s, (const TI*)qkv, row_stride, bias, \
             (const TW*)q_w, (const TW*)k_w, norm_mode, eps, positions, cos_t, sin_t, rot, interleaved, slot_of_token, (TA*)cache, \
-            (TA*)q_out, Hq, Hkv, Hv, dk, dv, has_kv, page_size)); } while (0)
+            (TA*)q_out, Hq, Hkv, Hv, dk, dv, has_kv, page_size, cv)); } while (0)
     if (act_dtype == RI_BF16) {
         if (in_dtype == RI_BF16) { if (w_dtype == RI_BF16) RI_QP(bf16, bf16, bf16); else RI_QP(bf16, bf16, float); }
         else { if (w_dtype == RI_BF16) RI_QP(float, bf16, bf16); else RI_QP(float, bf16, float); }

@@ -10,7 +10,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..parts import (attention, attention_variants, experts, ffn, hyper, linear_attention, norm, parallel,  # noqa: F401
-                     recurrent_unit, rope, short_conv, stem_tail)  # (registers the built-in parts)
+                     recurrent_unit, rope, short_conv, state_space, stem_tail)  # (registers the built-in parts)
 from ..parts.base import EMBEDDINGS, HEADS, NORMS, BuildContext, CacheNeed, ParamDecl, StepContext, StepIndex
 from ..parts.block import Block, Hidden
 from ..parts.spec import ModelSpec

@@ -97,13 +97,14 @@ def rope_scatter(qkv: torch.Tensor, positions: torch.Tensor, cos: Optional[torch
                                    max(page, 1), stream_ptr()), "rope_scatter")
 
 
-def silu_mul(gu: torch.Tensor, out: torch.Tensor) -> None:
+def silu_mul(gu: torch.Tensor, out: torch.Tensor, gelu: bool = False) -> None:
+    """gu [T, 2I], gates first: out = silu(gate) * up, or with `gelu` the tanh form of gelu(gate) * up."""
     require_cuda(gu, out)
     _contig(gu, "gu"); _contig(out, "out")
     T, two_i = gu.shape
     if two_i % 2 or out.shape != (T, two_i // 2) or out.dtype != gu.dtype:
         raise KernelError("silu_mul: gu is [T, 2I], out [T, I] of the same dtype")
-    check(L.core().ri_silu_mul(_p(gu), _p(out), dtype_code(gu.dtype), T, two_i // 2, stream_ptr()),
+    check(L.core().ri_silu_mul(_p(gu), _p(out), dtype_code(gu.dtype), T, two_i // 2, 1 if gelu else 0, stream_ptr()),
           "silu_mul")
 
 
@@ -124,6 +125,7 @@ def gemm_f32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
 # ------------------------------------------------------------ tcgen05 bf16 matrix product
 EPI_BF16, EPI_F32, EPI_SILU, EPI_RESIDUAL = 0, 1, 2, 3
 EPI_RELU2 = 5             # max(x, 0)^2 of the fp32 sums, stored bf16
+EPI_GELU = 6              # EPI_SILU's pairs with the tanh form of gelu in place of silu
 _tc_state = {}
 _TC_WORKSPACE_FLOATS = 8 << 20
 _TC_COUNTERS = 1 << 14
@@ -191,7 +193,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int =
     """out = x[M,K] @ w[N,K]^T on the tcgen05 tensor cores, bf16 inputs, fp32 accumulation.
     epilogue: EPI_BF16 / EPI_F32 store into out [M,N]; EPI_SILU stores silu(gate)*up into
     out [M,N/2] for a weight whose rows alternate gate_j, up_j; EPI_RESIDUAL adds into the
-    fp32 out [M,N]; EPI_RELU2 stores max(x, 0)^2 as bf16."""
+    fp32 out [M,N]; EPI_RELU2 stores max(x, 0)^2 as bf16; EPI_GELU is EPI_SILU with gelu_tanh(gate)*up."""
     require_cuda(x, w, out)
     if not gemm_tc_supports(x, w):
         raise KernelError("gemm_tc: contiguous, 16-byte aligned bfloat16 x [M,K] and w [N,K] with K a multiple of 8")
@@ -199,9 +201,10 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int =
     N = w.shape[0]
     if w.shape[1] != Kd or out.stride(1) != 1:
         raise KernelError(f"gemm_tc: shapes x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
-    cols = N // 2 if epilogue == EPI_SILU else N
-    want = torch.bfloat16 if epilogue in (EPI_BF16, EPI_SILU, EPI_RELU2) else torch.float32
-    if out.dtype != want or out.shape != (M, cols) or (epilogue == EPI_SILU and N % 2):
+    pairs = epilogue in (EPI_SILU, EPI_GELU)
+    cols = N // 2 if pairs else N
+    want = torch.bfloat16 if pairs or epilogue in (EPI_BF16, EPI_RELU2) else torch.float32
+    if out.dtype != want or out.shape != (M, cols) or (pairs and N % 2):
         raise KernelError(f"gemm_tc: out must be {want} [{M}, {cols}] for epilogue {epilogue}")
     plan = plan or gemm_tc_plan(M, N, Kd, num_sms, epilogue)
     swap, bn, splits = plan[:3]
@@ -398,7 +401,7 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, blo
                     scale: float, window: Optional[int], block: Optional[int] = None,
                     value_dim: Optional[int] = None, sink: bool = False, softcap: Optional[float] = None,
                     sink_values: Optional[torch.Tensor] = None, maps: int = 1, value_in_key: bool = False,
-                    slopes: Optional[torch.Tensor] = None) -> None:
+                    slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> None:
     """q [T, >=Hq*hd] (may be a column view of the qkv buffer), out [T, Hq*vd].  `block`: a query
     sees only the keys of its own block of that many positions (counted from 0).  `value_dim`:
     size of a value where it is not the keys'; the cache is then [pages, Hkv*page*(hd+vd)].  `sink`:
@@ -409,9 +412,10 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, blo
     heads, and the cache holds Hkv*m key heads ([kv head][map]).  `value_in_key`: a key's value is
     its own first `value_dim` channels, and the cache holds keys only.  `slopes` (fp32 [Hq]): a linear
     distance bias, slopes[h] * (query position - key position) taken off head h's scores after scale
-    and cap.  `out` may be fp32 whatever the cache's dtype."""
-    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_q0, sink_values, slopes)
-    _slopes_ok(slopes, num_heads)
+    and cap.  `bias` (fp32 [Hq, n]): bias[h, min(query position - key position, n - 1)] added to head h's
+    scores after scale and cap.  `out` may be fp32 whatever the cache's dtype."""
+    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_q0, sink_values, slopes, bias)
+    _slopes_ok(slopes, num_heads, bias)
     for t, n in ((block_table, "block_table"), (cu_q, "cu_q"), (kv_len, "kv_len"),
                  (tile_entry, "tile_entry"), (tile_q0, "tile_q0")):
         _i32(t, n)
@@ -425,11 +429,14 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, blo
                                     int(window) if window else 0, int(block) if block else 0, 1 if sink else 0,
                                     float(softcap) if softcap else 0.0, _p(sink_values), int(maps),
                                     1 if value_in_key else 0, 1 if out.dtype == torch.float32 else 0, _p(slopes),
-                                    stream_ptr()),
+                                    _p(bias), bias.shape[1] if bias is not None else 0, stream_ptr()),
           "attention_plain")
 
 
-def _slopes_ok(slopes: Optional[torch.Tensor], num_heads: int) -> None:
+def _slopes_ok(slopes: Optional[torch.Tensor], num_heads: int, bias: Optional[torch.Tensor] = None) -> None:
+    if bias is not None and (bias.dtype != torch.float32 or bias.dim() != 2 or bias.shape[0] != num_heads or bias.shape[1] < 1
+                             or not bias.is_contiguous()):
+        raise KernelError("attention: bias is contiguous fp32 [heads, distances]")
     if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != num_heads or not slopes.is_contiguous()):
         raise KernelError("attention: slopes is fp32 [heads]")
 
@@ -462,13 +469,13 @@ def attention_single(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                      block: Optional[int] = None, value_dim: Optional[int] = None, sink: bool = False,
                      splits: int = 1, part: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
                      sink_values: Optional[torch.Tensor] = None, maps: int = 1, value_in_key: bool = False,
-                     slopes: Optional[torch.Tensor] = None) -> None:
+                     slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> None:
     """Attention of the entries that bring one token (`entry_list`, int32; -1 skips): fp32 arithmetic, a kv
     head's keys and values read once for all its query heads.  Arguments as `attention_plain`.  `splits` > 1
     cuts every entry's keys into that many ranges, a CTA each, joined by a second launch through `part`
     (fp32, `attention_single_scratch_floats` long)."""
-    require_cuda(q, out, cache, block_table, cu_q, kv_len, entry_list, part, sink_values, slopes)
-    _slopes_ok(slopes, num_heads)
+    require_cuda(q, out, cache, block_table, cu_q, kv_len, entry_list, part, sink_values, slopes, bias)
+    _slopes_ok(slopes, num_heads, bias)
     if splits > 1 and (part is None or part.dtype != torch.float32 or not part.is_contiguous() or
                        part.numel() < attention_single_scratch_floats(entry_list.numel(), num_heads, value_dim or head_dim, splits)):
         raise KernelError("attention_single: the scratch for the key ranges is too small")
@@ -484,7 +491,7 @@ def attention_single(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                                      int(splits), _p(part) if splits > 1 else None,
                                      float(softcap) if softcap else 0.0, _p(sink_values), int(maps),
                                      1 if value_in_key else 0, 1 if out.dtype == torch.float32 else 0, _p(slopes),
-                                     stream_ptr()),
+                                     _p(bias), bias.shape[1] if bias is not None else 0, stream_ptr()),
           "attention_single", 2 if splits > 1 else 1)
 
 
@@ -507,14 +514,15 @@ def attention_rows(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
                    num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: Optional[int],
                    value_dim: Optional[int] = None, sink: bool = False, softcap: Optional[float] = None,
                    sink_values: Optional[torch.Tensor] = None, maps: int = 1, value_in_key: bool = False,
-                   splits: int = 1, part: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> None:
+                   splits: int = 1, part: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
+                   bias: Optional[torch.Tensor] = None, block: Optional[int] = None) -> None:
     """`attention_plain` on the tensor cores for a bf16 cache: the scores are fp32 sums of products of bf16 q and
     k, cap, mask and softmax are fp32, and the softmax weights meet the bf16 values unrounded (three bf16 pieces a
-    weight).  Arguments as there, without `block`; tiles hold `attention_rows_tokens_per_tile` tokens.  `splits` > 1
+    weight).  Arguments as there; tiles hold `attention_rows_tokens_per_tile` tokens.  `splits` > 1
     cuts every tile's keys into that many ranges, a CTA each, joined by a second launch through `part` (fp32,
     `attention_rows_scratch_floats` long): for few tiles over many keys."""
-    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_tok0, sink_values, part, slopes)
-    _slopes_ok(slopes, num_heads)
+    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_tok0, sink_values, part, slopes, bias)
+    _slopes_ok(slopes, num_heads, bias)
     for t, n in ((block_table, "block_table"), (cu_q, "cu_q"), (kv_len, "kv_len"),
                  (tile_entry, "tile_entry"), (tile_tok0, "tile_tok0")):
         _i32(t, n)
@@ -532,7 +540,8 @@ def attention_rows(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
         _p(kv_len), _p(tile_entry), _p(tile_tok0), tile_entry.numel(), num_heads, num_kv_heads, page_size, float(scale),
         int(window) if window else 0, 1 if sink else 0, float(softcap) if softcap else 0.0, _p(sink_values), int(maps),
         1 if value_in_key else 0, 1 if out.dtype == torch.float32 else 0, int(splits), _p(part) if splits > 1 else None,
-        _p(slopes), stream_ptr()), "attention_rows", 2 if splits > 1 else 1)
+        _p(slopes), _p(bias), bias.shape[1] if bias is not None else 0, int(block) if block else 0, stream_ptr()),
+        "attention_rows", 2 if splits > 1 else 1)
 
 
 def attention_rows_ctas_per_sm(head_dim: int, value_dim: int, value_in_key: bool, out_dtype: torch.dtype) -> int:
@@ -632,13 +641,16 @@ def short_conv_max_taps() -> int:
 
 def short_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor,
                cu_q: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor, n_entries: int, max_q_len: int,
-               residual: bool, in_bias: Optional[torch.Tensor] = None) -> None:
+               residual: bool, in_bias: Optional[torch.Tensor] = None, silu: bool = False,
+               steps: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor, torch.Tensor, torch.Tensor]] = None) -> None:
     """A causal convolution over time on every channel, continued from a state: out[t] = (x[t] if residual) + bias +
     sum_j weight[:, j] * x[t - taps + 1 + j] over each entry's tokens (x [T, C], may be a column view; weight fp32
     [C, taps]); the taps - 1 inputs before an entry's first token come from state[slot] (fp32 [slots, taps - 1, C],
     oldest first) and the entry's last taps - 1 inputs go back there.  `in_bias` (fp32 [C]) is added to every input
-    first (the state holds the sums)."""
-    require_cuda(x, weight, bias, state, cu_q, state_slots, out, in_bias)
+    first (the state holds the sums).  `silu`: the activation after the bias.  `steps` (raw, dt_bias, a_log, dt, decay):
+    raw [T, H] are the columns of x's rows right behind x's own; dt = softplus(raw + dt_bias) and decay =
+    exp(-exp(a_log) * dt) (both fp32 [T, H]; dt_bias and a_log fp32 [H]) are made in the same launch."""
+    require_cuda(x, weight, bias, state, cu_q, state_slots, out, in_bias, *(steps or ()))
     _f32_vec(in_bias, x.shape[1], "short_conv: in_bias")
     _i32(cu_q, "cu_q"); _i32(state_slots, "state_slots")
     T, C = x.shape
@@ -650,9 +662,22 @@ def short_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
     _f32_vec(bias, C, "short_conv: bias")
     if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (taps - 1, C):
         raise KernelError("short_conv: state is contiguous fp32 [slots, taps - 1, C]")
+    dtb = alog = dt = decay = None
+    H = 0
+    if steps is not None:
+        raw, dtb, alog, dt, decay = steps
+        H = raw.shape[1]
+        if (raw.dtype != x.dtype or raw.shape[0] != T or raw.stride() != x.stride()
+                or raw.data_ptr() != x.data_ptr() + C * x.element_size()):
+            raise KernelError("short_conv: the step sizes are the columns right behind x's")
+        _f32_vec(dtb, H, "short_conv: dt_bias"); _f32_vec(alog, H, "short_conv: a_log")
+        for t in (dt, decay):
+            if t.dtype != torch.float32 or t.shape != (T, H) or not t.is_contiguous():
+                raise KernelError("short_conv: dt and decay are contiguous fp32 [T, H]")
     check(L.core().ri_short_conv(_p(x), dtype_code(x.dtype), x.stride(0), _p(weight), _p(bias), _p(state), _p(cu_q),
                                  _p(state_slots), _p(out), dtype_code(out.dtype), out.stride(0), int(n_entries),
-                                 int(max_q_len), C, taps, 1 if residual else 0, _p(in_bias), stream_ptr()), "short_conv")
+                                 int(max_q_len), C, taps, 1 if residual else 0, _p(in_bias), 1 if silu else 0, _p(dtb),
+                                 _p(alog), _p(dt), _p(decay), H, stream_ptr()), "short_conv")
 
 
 def rglru_gates(u: torch.Tensor, wa: torch.Tensor, wi: torch.Tensor, ba: torch.Tensor, bi: torch.Tensor,
@@ -897,14 +922,18 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight: Optio
                 cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rotary_dim: int, interleaved: bool,
                 slot_of_token: Optional[torch.Tensor], cache: Optional[torch.Tensor], q_out: torch.Tensor,
                 num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, has_kv: bool,
-                value_heads: Optional[int] = None) -> None:
+                value_heads: Optional[int] = None,
+                conv: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None) -> None:
     """qkv [T, Hq*hd (+ Hkv*hd + Hkv*vd when `has_kv`)]: add `bias` (fp32), norm q and k (`norm_mode` 0: not;
     1: every head by its own root mean square, weights [hd]; 2: all heads at once, weights [Hq*hd] and
     [Hkv*hd]), rotate the first `rotary_dim` channels of every head (pairs (2i, 2i+1) when `interleaved`, else
     (i, i + rotary_dim/2)), write q into q_out [T, Hq*hd] and k, v into the cache at slot_of_token[t].
     `value_heads`: heads of v where they are fewer than the heads of k (`num_kv_heads` then counts the key
-    heads: kv heads times the attention maps of a head).  qkv may be the leading columns of wider rows."""
-    require_cuda(qkv, bias, q_weight, k_weight, positions, cos, sin, slot_of_token, cache, q_out)
+    heads: kv heads times the attention maps of a head).  qkv may be the leading columns of wider rows.  `conv`
+    (weight fp32 [columns, taps], state fp32 [slots, taps - 1, columns], state_slots int32 [T]), for a step in which
+    row t is the one token of entry t: every column first passes the short convolution as `short_conv` computes it,
+    its earlier inputs from state[state_slots[t]], which the new input is shifted into."""
+    require_cuda(qkv, bias, q_weight, k_weight, positions, cos, sin, slot_of_token, cache, q_out, *(conv or ()))
     _i32(positions, "positions"); _i32(slot_of_token, "slot_of_token")
     T = qkv.shape[0]
     Hv = value_heads or num_kv_heads
@@ -934,25 +963,43 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight: Optio
         if cache.dtype != q_out.dtype:
             raise KernelError("qkv_prepare: the cache has q_out's dtype")
         page = paged_cache_page_size(cache, Hv, head_dim, value_dim, num_kv_heads // Hv)
+    cw = cs = cslots = None
+    taps = 0
+    if conv is not None:
+        cw, cs, cslots = conv
+        taps = cw.shape[1]
+        _i32(cslots, "conv slots")
+        if cw.dtype != torch.float32 or cw.shape[0] != cols or not cw.is_contiguous() or cs.dtype != torch.float32 \
+                or not cs.is_contiguous() or tuple(cs.shape[1:]) != (taps - 1, cols) or cslots.numel() < T:
+            raise KernelError("qkv_prepare: conv is (fp32 [columns, taps], fp32 [slots, taps - 1, columns], int32 [T])")
     check(L.core().ri_qkv_prepare(_p(qkv), dtype_code(qkv.dtype), qkv.stride(0), _p(bias), _p(q_weight), _p(k_weight),
                                   dtype_code(ws[0].dtype) if ws else 0, int(norm_mode), float(eps), _p(positions),
                                   _p(cos), _p(sin), int(rotary_dim), 1 if interleaved else 0, _p(slot_of_token), _p(cache),
                                   _p(q_out), dtype_code(q_out.dtype), T, num_heads, num_kv_heads, head_dim, value_dim,
-                                  1 if has_kv else 0, page, Hv, stream_ptr()), "qkv_prepare")
+                                  1 if has_kv else 0, page, Hv, _p(cw), _p(cs), _p(cslots), int(taps), stream_ptr()), "qkv_prepare")
 
 
 # ------------------------------------------------------------------------ routed experts
+_ROUTER_SCORES = {"sigmoid": 0, "softmax_chosen": 1, "softmax": 2}
+
+
 def moe_route(z: Optional[torch.Tensor], correction: Optional[torch.Tensor], top: int, n_groups: int, keep: int, renorm: bool,
               ids: torch.Tensor, weights: torch.Tensor, counts: torch.Tensor, x: Optional[torch.Tensor] = None,
-              router: Optional[torch.Tensor] = None, score: str = "sigmoid") -> None:
+              router: Optional[torch.Tensor] = None, score: str = "sigmoid", group_score: str = "top2",
+              renorm_eps: float = 0.0, gate: Optional[torch.Tensor] = None) -> None:
     """The `top` experts of every token (ids int32 [T, top]) and their weights (fp32 [T, top]) from router logits:
     either z [T, E] fp32 is given, or x [T, d] and the router's matrix (fp32 [E, d]) and the kernel forms z = x W^T
     itself in fp32.  Scores sigmoid(z), chosen by score + correction among the experts of the `keep` best of
     `n_groups` groups (0: no groups).  With `score` "softmax_chosen" the scores are the logits themselves and the
-    weights the softmax of the chosen logits among themselves.  counts (int32 [E]) gets one added per choice."""
-    if score not in ("sigmoid", "softmax_chosen"):
-        raise KernelError(f"moe_route: score {score!r}")
-    require_cuda(z, correction, ids, weights, counts, x, router)
+    weights the softmax of the chosen logits among themselves; with "softmax" the scores are the softmax over all
+    experts.  `group_score`: a group's score is the sum of its two largest ("top2") or its largest ("max").
+    `renorm`: the weights are divided by their sum + `renorm_eps`.  `gate` (fp32 [T], with x): the router's matrix has one row
+    more, [E + 1, d], and gate = sigmoid(x . that row).  counts (int32 [E]) gets one added per choice."""
+    if score not in _ROUTER_SCORES or group_score not in ("top2", "max"):
+        raise KernelError(f"moe_route: score {score!r}, group score {group_score!r}")
+    require_cuda(z, correction, ids, weights, counts, x, router, gate)
+    if gate is not None and (x is None or gate.dtype != torch.float32 or gate.numel() != ids.shape[0]):
+        raise KernelError("moe_route: gate is fp32 [T] and goes with the router's input")
     E = counts.numel()
     T = ids.shape[0]
     _contig(ids, "ids"); _contig(weights, "weights"); _i32(ids, "ids"); _i32(counts, "counts")
@@ -963,7 +1010,7 @@ def moe_route(z: Optional[torch.Tensor], correction: Optional[torch.Tensor], top
     d = 0
     if x is not None:
         d = x.shape[1]
-        if router is None or router.dtype != torch.float32 or tuple(router.shape) != (E, d) or not router.is_contiguous() \
+        if router is None or router.dtype != torch.float32 or tuple(router.shape) != (E + (gate is not None), d) or not router.is_contiguous() \
                 or not x.is_contiguous() or x.shape[0] != T:
             raise KernelError("moe_route: x is contiguous [T, d] and the router's matrix fp32 [E, d]")
     if weights.dtype != torch.float32 or ids.shape != (T, top) or weights.shape != (T, top) \
@@ -971,7 +1018,8 @@ def moe_route(z: Optional[torch.Tensor], correction: Optional[torch.Tensor], top
         raise KernelError("moe_route: correction fp32 [E], ids int32 and weights fp32 [T, top], counts [E]")
     check(L.core().ri_moe_route(_p(z), _p(x), dtype_code(x.dtype) if x is not None else 0, _p(router), d, _p(correction), T, E,
                                 int(top), int(n_groups), int(keep), 1 if renorm else 0, _p(ids), _p(weights), _p(counts),
-                                1 if score == "softmax_chosen" else 0, stream_ptr()), "moe_route")
+                                _ROUTER_SCORES[score], 1 if group_score == "max" else 0, float(renorm_eps), _p(gate),
+                                stream_ptr()), "moe_route")
 
 
 def moe_sort(ids: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor, order: torch.Tensor, place: torch.Tensor) -> None:
@@ -1048,9 +1096,11 @@ def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets
 
 
 def moe_combine(Y: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, shared: Optional[torch.Tensor],
-                out: torch.Tensor, counts: torch.Tensor) -> None:
-    """out[t] = sum_j weights[t, j] * Y[place[t * top + j]] (+ shared[t]); counts is put back to zero."""
-    require_cuda(Y, place, weights, shared, out, counts)
+                out: torch.Tensor, counts: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
+    """out[t] = sum_j weights[t, j] * Y[place[t * top + j]] (+ gate[t] * shared[t]; gate fp32 [T], None: 1); counts is put
+    back to zero."""
+    require_cuda(Y, place, weights, shared, out, counts, gate)
+    _f32_vec(gate, out.shape[0], "moe_combine: gate")
     T, top = weights.shape
     d = Y.shape[1]
     _contig(Y, "Y"); _contig(out, "out"); _contig(weights, "weights"); _i32(place, "place"); _i32(counts, "counts")
@@ -1059,7 +1109,7 @@ def moe_combine(Y: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, sha
         raise KernelError("moe_combine: Y fp32 [T*top, d], weights fp32 [T, top], shared and out [T, d]")
     check(L.core().ri_moe_combine(_p(Y), _p(place), _p(weights), _p(shared),
                                   dtype_code(shared.dtype) if shared is not None else 0, _p(out), dtype_code(out.dtype),
-                                  T, top, d, _p(counts), counts.numel(), stream_ptr()), "moe_combine")
+                                  T, top, d, _p(counts), counts.numel(), _p(gate), stream_ptr()), "moe_combine")
 
 
 GATE_SILU, GATE_SIGMOID = 0, 1
@@ -1190,6 +1240,42 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.T
                                         stream_ptr()), "decay_scan")
 
 
+def head_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, q_scale: float, out: torch.Tensor,
+              state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, entries: int, num_heads: int, key_dim: int,
+              value_dim: int, gain: Optional[torch.Tensor] = None, key_heads: Optional[int] = None,
+              rotation: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor, int, bool]] = None) -> None:
+    """Linear attention with one decay a head, over every entry's tokens in order, from and into state[slot]:
+    S = decay_h S + k (gain_h v)^T, out = S^T (q * q_scale).  `decay` fp32 [H] (fixed) or [T, H]; `gain` fp32 [T, H] or
+    None (1); head h reads key and query head h // (H / key_heads) of q, k [T, key_heads*dk]; v [T, H*dv]; column views
+    allowed.  State as `gated_scan`.  `rotation` (positions int32 [T], cos, sin fp32 [positions, rot/2], rot, interleaved):
+    keys and queries are rotated on the way in; only for a step in which every entry brings one token (T == entries)."""
+    require_cuda(q, k, v, decay, out, state, cu_q, state_slots, gain, *(rotation[:3] if rotation else ()))
+    T, H, dk, dv = q.shape[0], num_heads, key_dim, value_dim
+    G = key_heads or H
+    if H % G:
+        raise KernelError("head_scan: heads are a multiple of key heads")
+    _scan_common(state, out, cu_q, state_slots, T, H, dk, dv, "head_scan")
+    _cols(q, T, G * dk, q.dtype, "head_scan: q"); _cols(k, T, G * dk, q.dtype, "head_scan: k")
+    _cols(v, T, H * dv, q.dtype, "head_scan: v")
+    if decay.dtype != torch.float32 or not decay.is_contiguous() or tuple(decay.shape) not in ((H,), (T, H)):
+        raise KernelError("head_scan: decay is contiguous fp32 [H] or [T, H]")
+    if gain is not None and (gain.dtype != torch.float32 or not gain.is_contiguous() or gain.shape != (T, H)):
+        raise KernelError("head_scan: gain is contiguous fp32 [T, H]")
+    pos = cos = sin = None
+    rot, inter = 0, False
+    if rotation is not None:
+        pos, cos, sin, rot, inter = rotation
+        _i32(pos, "positions")
+        if T != int(entries) or cos.dtype != torch.float32 or cos.shape[1] != rot // 2 or sin.shape != cos.shape \
+                or not cos.is_contiguous() or not sin.is_contiguous():
+            raise KernelError("head_scan: rotation goes with single tokens; cos/sin are fp32 [positions, rot/2]")
+    check(L.recurrent(dk).ri_head_scan(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(decay),
+                                       H if decay.dim() == 2 else 0, _p(gain), H if gain is not None else 0,
+                                       dtype_code(q.dtype), float(q_scale), _p(out), _p(state), _p(cu_q), _p(state_slots),
+                                       int(entries), H, dv, H // G, _p(pos), _p(cos), _p(sin), int(rot), 1 if inter else 0,
+                                       1 if T == int(entries) else 0, stream_ptr()), "head_scan")
+
+
 def delta_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, za: torch.Tensor, za_bias: Optional[torch.Tensor],
                zw: torch.Tensor, zw_bias: Optional[torch.Tensor], decay_rate: float, unit_eps: float,
                out: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, entries: int,
@@ -1218,6 +1304,80 @@ def delta_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, za: torch.Tens
                                         _p(unit[1]), H * dk, dtype_code(r.dtype), _p(out), _p(state), _p(cu_q),
                                         _p(state_slots), int(entries), H, dv, 1 if T == int(entries) else 0,
                                         stream_ptr()), "delta_scan")
+
+
+# --------------------------------------------- blocks that norm a sublayer's output, and their mixers
+def norm_add(h: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tensor, eps: float, act: Optional[torch.Tensor],
+             experts: Optional[Tuple] = None) -> None:
+    """h (fp32 [T, d]) += rms(y) * weight, in place; `act` (may be None) gets the new h rounded to its dtype.  `weight` fp32
+    [d], or one number for all channels.  y [T, d]; or None with `experts` (Y, place, weights, shared, gate, counts), the
+    arguments of `moe_combine`: y is then the weighted sum of a token's experts, formed in the same launch, and counts is
+    put back to zero."""
+    require_cuda(h, y, weight, act, *(experts or ()))
+    _contig(h, "h"); _contig(weight, "weight")
+    T, d = h.shape
+    if h.dtype != torch.float32 or weight.dtype != torch.float32 or weight.numel() not in (1, d):
+        raise KernelError("norm_add: h is fp32 [T, d], weight fp32 of one number or d")
+    if act is not None and (act.shape != h.shape or not act.is_contiguous()):
+        raise KernelError("norm_add: act has h's shape")
+    if (y is None) == (experts is None):
+        raise KernelError("norm_add: give the sublayer's output or the experts' rows, not both")
+    Y = place = wts = shared = gate = counts = None
+    top = 0
+    if y is not None:
+        if y.shape != h.shape or not y.is_contiguous():
+            raise KernelError("norm_add: y has h's shape")
+    else:
+        Y, place, wts, shared, gate, counts = experts
+        top = wts.shape[1]
+        _i32(place, "place"); _i32(counts, "counts")
+        for t in (Y, wts, shared, gate):
+            if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+                raise KernelError("norm_add: the experts' rows, weights, shared rows and gate are contiguous fp32")
+        if Y.shape != (T * top, d) or wts.shape[0] != T or place.numel() != T * top or (shared is not None and shared.shape != (T, d)) \
+                or (gate is not None and gate.numel() != T):
+            raise KernelError("norm_add: Y [T*top, d], weights [T, top], place [T*top], shared [T, d], gate [T]")
+    check(L.core().ri_norm_add(_p(h), _p(y), dtype_code(y.dtype) if y is not None else 0, _p(weight), 1 if weight.numel() == 1 else 0,
+                               float(eps), _p(act), dtype_code(act.dtype) if act is not None else 0, T, d, _p(Y), _p(place), _p(wts),
+                               _p(shared), _p(gate), int(top), _p(counts), counts.numel() if counts is not None else 0,
+                               stream_ptr()), "norm_add")
+
+
+def rotate_cols(x: torch.Tensor, positions: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, num_heads: int, head_dim: int,
+                rotary_dim: int, interleaved: bool = False) -> None:
+    """x fp32 [T, heads*head_dim] (may be a column view): the first `rotary_dim` channels of every head turn in place by the
+    angles of the token's position; pairs (i, i + rotary_dim/2), or (2i, 2i+1) when `interleaved`."""
+    require_cuda(x, positions, cos, sin)
+    _i32(positions, "positions")
+    _cols(x, x.shape[0], num_heads * head_dim, torch.float32, "rotate_cols: x")
+    for t in (cos, sin):
+        if t.dtype != torch.float32 or t.shape[1] != rotary_dim // 2 or not t.is_contiguous():
+            raise KernelError("rotate_cols: cos/sin are fp32 [positions, rotary_dim/2]")
+    check(L.core().ri_rotate_cols(_p(x), x.stride(0), _p(positions), _p(cos), _p(sin), x.shape[0], num_heads, head_dim,
+                                  int(rotary_dim), 1 if interleaved else 0, stream_ptr()), "rotate_cols")
+
+
+def part_norm_gate(o: torch.Tensor, z: torch.Tensor, weight: Optional[torch.Tensor], parts: int, eps: float, gate_first: bool,
+                   out: torch.Tensor, skip: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
+    """A row of o (fp32 [T, n]) in `parts` equal parts, each normed by its own root mean square.  With y = o (+ D[channel's
+    head] * x for `skip` (D fp32 [heads], x fp32 [T, n])):  out = rms(y * silu(z)) * weight when `gate_first`, else
+    out = rms(y) * weight * silu(z).  z and x fp32 (may be column views), weight fp32 [n] or None."""
+    D, x = skip if skip is not None else (None, None)
+    require_cuda(o, z, weight, out, D, x)
+    _contig(o, "o"); _contig(out, "out")
+    T, n = o.shape
+    _f32_vec(weight, n, "part_norm_gate: weight")
+    if o.dtype != torch.float32 or out.shape != o.shape or parts <= 0 or n % parts:
+        raise KernelError("part_norm_gate: o is fp32 [T, n], out has its shape, parts divide n")
+    _cols(z, T, n, torch.float32, "part_norm_gate: z")
+    if D is not None:
+        _cols(x, T, n, torch.float32, "part_norm_gate: x")
+        if n % D.numel():
+            raise KernelError("part_norm_gate: the heads of D divide the row")
+        _f32_vec(D, D.numel(), "part_norm_gate: D")
+    check(L.core().ri_part_norm_gate(_p(o), _p(x), x.stride(0) if x is not None else 0, _p(D), n // D.numel() if D is not None else 1,
+                                     _p(z), z.stride(0), _p(weight), float(eps), 1 if gate_first else 0, _p(out),
+                                     dtype_code(out.dtype), T, int(parts), n // int(parts), stream_ptr()), "part_norm_gate")
 
 
 # ------------------------------------------------- blocks that norm after the sum, and their mixers

@@ -23,7 +23,7 @@ _SIGNATURES = {
     "ri_add_rmsnorm": [_P, _P, _P, _I, _F, _P, _I, _P, _I, _I, _P],
     "ri_residual_add": [_P, _P, _I, _L, _P],
     "ri_rope_scatter": [_P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-    "ri_silu_mul": [_P, _P, _I, _I, _I, _P],
+    "ri_silu_mul": [_P, _P, _I, _I, _I, _I, _P],
     "ri_gemm_f32": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _P],
     "ri_argmax": [_P, _I, _I, _I, _P, _P, _P, _P],
     "ri_decode_feedback": [_P, _P, _I, _P, _P, _I, _P, _P, _P],
@@ -42,10 +42,10 @@ _SIGNATURES = {
     "ri_attention_single": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P],
     "ri_embed_rmsnorm": [_P, _P, _I, _P, _I, _F, _P, _I, _I, _I, _P],
     "ri_hyper_collect": [_P, _I, _P, _I, _P, _P, _P, _P, _I, _F, _P, _I, _P, _I, _I, _I, _I, _P],
-    "ri_qkv_prepare": [_P, _I, _I, _P, _P, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
-    "ri_attention_plain_ex": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P],
-    "ri_attention_single_ex": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _F, _P, _I, _I, _I, _P, _P],
-    "ri_attention_rows": [_P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _P, _I, _I, _I, _I, _P, _P, _P],
+    "ri_qkv_prepare": [_P, _I, _I, _P, _P, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P],
+    "ri_attention_plain_ex": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _F, _P, _I, _I, _I, _P, _P, _I, _P],
+    "ri_attention_single_ex": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _F, _P, _I, _I, _I, _P, _P, _I, _P],
+    "ri_attention_rows": [_P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P],
     "ri_attention_rows_tokens_per_tile": [_I, _I, _I],
     "ri_attention_rows_ctas_per_sm": [_I, _I],
     "ri_embed_scaled": [_P, _P, _I, _F, _P, _I, _I, _I, _P],
@@ -56,12 +56,12 @@ _SIGNATURES = {
     "ri_latent_prepare": [_P, _I, _I, _P, _I, _F, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P],
     "ri_bias_rows": [_P, _I, _P, _I, _I, _I, _P],
     "ri_activation_cols": [_P, _I, _I, _I, _I, _I, _P],
-    "ri_moe_route": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P],
+    "ri_moe_route": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _F, _P, _P],
     "ri_moe_sort": [_P, _P, _I, _I, _P, _P, _P, _P],
     "ri_moe_product": [_P, _I, _I, _P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "ri_moe_gather": [_P, _P, _I, _P, _I, _I, _P],
     "ri_gemm_tc_grouped": [_P, _P, _I, _I, _I, _P, _I, _I, _P, _I, _P, _F, _F, _P],
-    "ri_moe_combine": [_P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P, _I, _P],
+    "ri_moe_combine": [_P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P, _I, _P, _P],
     "ri_attention_single_supports": [_I, _I],
     "ri_embed_sinusoid": [_P, _P, _P, _I, _P, _P, _I, _I, _I, _P],
     "ri_sandwich_norm": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _F, _P],
@@ -72,19 +72,23 @@ _SIGNATURES = {
     "ri_gated_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     "ri_delta_scan": [_P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     "ri_rms_sandwich": [_P, _I, _P, _I, _I, _P, _P, _P, _L, _I, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P, _P, _P, _I, _P],
-    "ri_short_conv": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "ri_short_conv": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P],
     "ri_rglru_gates": [_P, _I, _P, _P, _I, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P],
     "ri_rglru_step": [_P, _I, _P, _P, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P],
     "ri_rglru_scan": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P],
     "ri_sigmoid_gate": [_P, _I, _I, _P, _I, _I, _P, _I, _I, _I, _F, _P],
     "ri_softcap": [_P, _L, _F, _P],
     "ri_glu_pairs": [_P, _P, _I, _L, _I, _F, _F, _P],
+    "ri_head_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P],
+    "ri_norm_add": [_P, _P, _I, _P, _I, _F, _P, _I, _I, _I, _P, _P, _P, _P, _P, _I, _P, _I, _P],
+    "ri_rotate_cols": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+    "ri_part_norm_gate": [_P, _P, _I, _P, _I, _P, _I, _P, _F, _I, _P, _I, _I, _I, _I, _P],
     "ri_gated_decay": [_P, _P, _I, _F, _I, _I, _P],
     "ri_delta_prepare": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _F, _F, _P, _P, _I, _I, _I, _P],
 }
 
 _CORE_SOURCES = ["elementwise.cu", "gemm_f32.cu", "sampling.cu", "sequence_parts.cu", "stream_parts.cu",
-                 "mixture_parts.cu", "postnorm_parts.cu", "depth_parts.cu"]
+                 "mixture_parts.cu", "postnorm_parts.cu", "depth_parts.cu", "outnorm_parts.cu"]
 _loaded: Dict[str, ctypes.CDLL] = {}
 
 

@@ -19,9 +19,10 @@ from typing import Dict, Optional
 import torch
 
 from ..ops import kernels as K
-from .base import (BuildContext, Mixer, PagedKV, PagedLayerCache, ParamDecl, POSITIONS, StepContext,
-                   register_mixer, single_token_entries, token_tiles)
+from .base import (BuildContext, Mixer, PagedKV, PagedLayerCache, ParamDecl, StepContext, register_mixer,
+                   shared_position, single_token_entries, token_tiles)
 from .linear import Linear
+from .short_conv import ConvState
 from .spec import PartSpec
 
 
@@ -38,10 +39,10 @@ class PlainAttend:
     ROWS_MAX_SPLITS = 32        # of the tensor-core kernel
 
     def __init__(self, ctx: BuildContext, heads: int, kv_heads: int, head_dim: int, value_dim: int, maps: int = 1,
-                 value_in_key: bool = False, window: Optional[int] = None):
+                 value_in_key: bool = False, window: Optional[int] = None, block: Optional[int] = None):
         self.ctx = ctx
         self.Hq, self.Hkv, self.hd, self.vd, self.maps = heads, kv_heads, head_dim, value_dim, maps
-        self.value_in_key, self.window = value_in_key, window
+        self.value_in_key, self.window, self.block = value_in_key, window, block
         fast = (ctx.dtype == torch.bfloat16 and os.environ.get("RUSTINFER_B200_BLOCK_ATTENTION", "fast") != "plain")
         self.rows = fast and K.attention_rows_supports(head_dim, value_dim, value_in_key)
         group = heads // (kv_heads * maps)
@@ -76,7 +77,7 @@ class PlainAttend:
         return [self._tiles] if self._single is None else [self._single, self._tiles]
 
     def _span(self, max_kv_len: int) -> int:
-        return min(max_kv_len, self.window) if self.window else max_kv_len
+        return min([max_kv_len] + [n for n in (self.window, self.block) if n])
 
     def _splits(self, n_single: int, max_kv_len: int) -> int:
         want = -(-4 * self.ctx.num_sms // max(1, n_single * self.Hkv * self.maps))
@@ -88,28 +89,29 @@ class PlainAttend:
 
     def __call__(self, q: torch.Tensor, out: torch.Tensor, step: StepContext, cache: PagedLayerCache, scale: float,
                  softcap: Optional[float] = None, sink_values: Optional[torch.Tensor] = None,
-                 slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
         g = step.groups[cache.group]
         opts = dict(value_dim=self.vd, sink=sink_values is not None, softcap=softcap, sink_values=sink_values,
-                    maps=self.maps, value_in_key=self.value_in_key, slopes=slopes)
+                    maps=self.maps, value_in_key=self.value_in_key, slopes=slopes, bias=bias)
         if self._single is not None:
             (single,) = step.index(self._single)
             if single.numel() and self.fast_single:
                 K.attention_single(q, out, cache.kv, g.block_table, step.cu_q, step.kv_len, single, self.Hq, self.Hkv,
-                                   self.hd, scale, self.window, None, splits=self._splits(single.numel(), step.max_kv_len),
+                                   self.hd, scale, self.window, self.block, splits=self._splits(single.numel(), step.max_kv_len),
                                    part=self.part, **opts)
             elif single.numel():
                 K.attention_rows(q, out, cache.kv, g.block_table, step.cu_q, step.kv_len, single,
                                  self.zero_tok0[: single.numel()], self.Hq, self.Hkv, self.hd, scale, self.window,
-                                 splits=self._rows_splits(single.numel(), step.max_kv_len), part=self.part, **opts)
+                                 splits=self._rows_splits(single.numel(), step.max_kv_len), part=self.part,
+                                 block=self.block, **opts)
         tile_entry, tile_tok0 = step.index(self._tiles)
         if tile_entry.numel():
             if self.rows:
                 K.attention_rows(q, out, cache.kv, g.block_table, step.cu_q, step.kv_len, tile_entry, tile_tok0,
-                                 self.Hq, self.Hkv, self.hd, scale, self.window, **opts)
+                                 self.Hq, self.Hkv, self.hd, scale, self.window, block=self.block, **opts)
             else:
                 K.attention_plain(q, out, cache.kv, g.block_table, step.cu_q, step.kv_len, tile_entry, tile_tok0,
-                                  self.Hq, self.Hkv, self.hd, scale, self.window, None, **opts)
+                                  self.Hq, self.Hkv, self.hd, scale, self.window, self.block, **opts)
         return out
 
 
@@ -121,17 +123,6 @@ def project_out(o: Linear, y: torch.Tensor, add_to: Optional[torch.Tensor]) -> t
     if not o.add_into(y, add_to):
         K.residual_add(add_to, o(y, out_dtype=torch.float32))
     return add_to
-
-
-def _shared_position(ctx: BuildContext, spec: Optional[PartSpec]):
-    if spec is None:
-        return None
-    key = ("position", spec.key(), ctx.max_model_len)
-    if key not in ctx.shared:
-        part = POSITIONS.build(spec)
-        part.prepare(ctx)
-        ctx.shared[key] = part
-    return ctx.shared[key]
 
 
 @register_mixer("differential_attention")
@@ -197,7 +188,7 @@ class DifferentialAttention(Mixer):
     def prepare(self, ctx: BuildContext) -> None:
         super().prepare(ctx)
         self.attend = PlainAttend(ctx, 2 * self.H, self.G, self.hd, self.vd, maps=2, window=self.window)
-        self.position = _shared_position(ctx, self.position_spec)
+        self.position = shared_position(ctx, self.position_spec)
 
     def step_indices(self):
         return self.attend.step_indices()
@@ -308,7 +299,7 @@ class LatentAttention(Mixer):
     def prepare(self, ctx: BuildContext) -> None:
         super().prepare(ctx)
         self.attend = PlainAttend(ctx, self.H, 1, self.kd, self.rank, value_in_key=True)
-        self.position = _shared_position(ctx, PartSpec("rope", {
+        self.position = shared_position(ctx, PartSpec("rope", {
             "head_dim": self.rd, "rotary_dim": self.rd, "theta": self.rot_base, "scaling": None,
             "layout": self.rot_layout})) if self.rd else None
 
@@ -367,17 +358,44 @@ class LatentAttention(Mixer):
         return self.o(y, out_dtype=torch.float32)
 
 
+def distance_bucket(n: int, rows: int, far: float) -> int:
+    """The row of a table of `rows` that serves keys n positions back: a row a distance for the first half of the rows, then
+    buckets that widen by the logarithm and reach the last row at the distance `far`."""
+    half = rows // 2
+    if n < half:
+        return n
+    if half == 0 or far <= half:
+        return rows - 1
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
+
+
+def bucket_bias(table: torch.Tensor, far: float, reach: Optional[int] = None) -> torch.Tensor:
+    """table [rows, H] -> fp32 [H, n] on the table's device, the bias of every head by distance: entry n - 1 holds from there
+    on.  `reach`: no key is further back than that many positions less one."""
+    rows, dist = table.shape[0], [0]
+    while dist[-1] < rows - 1 and (reach is None or len(dist) < reach):
+        dist.append(distance_bucket(len(dist), rows, far))
+    index = torch.tensor(dist, dtype=torch.long, device=table.device)
+    return table.to(torch.float32)[index].t().contiguous()
+
+
 @register_mixer("distance_bias_attention")
 class DistanceBiasAttention(Mixer):
-    """Grouped-query attention without rotation, whose scores carry a linear distance bias:
+    """Grouped-query attention without rotation, whose scores carry a distance bias:
 
         score(i, j) = q_i . k_j * scale - slope_h * (i - j),    slope_h = 2^(-slope_exponent * (h + 1) / H)
+        or            q_i . k_j * scale + rel[bucket(i - j), h]   (`bias` "buckets"; see `distance_bucket`)
 
-    for head h of H, over the keys of a sliding window (None: every earlier key).  params: hidden_size, num_heads,
-    num_kv_heads, head_dim, value_dim, scale, window, slope_exponent (default 8), sink (the softmax's denominator
+    for head h of H, over the keys of a sliding window (None: every earlier key) and of the query's own block of `block`
+    positions (None: no blocks).  params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim, scale, window, block,
+    bias ("slopes", the default, or "buckets" with bias_far, the distance of the last row), slope_exponent (default 8),
+    conv_taps (None; else q, k and v pass a short causal convolution a channel right after their projection, weights
+    `q.conv` [channels, taps] and so on), qk_norm_eps (None; else one RMS norm over all heads of q and one over all of k,
+    weights `q.norm`, `k.norm` of those sizes, after the convolution), sink (the softmax's denominator
     holds exp(sink_h), a learned number per head with no key or value), head_gate (head h's output is multiplied
-    by sigmoid of the h-th of H numbers W_g x), tensor_names.  Tensors: q, k, v, o, and `sink` [H], `g` [H, hidden]
-    where asked for; no biases.  q, k, v and the gates are one product of the input; scores, softmax weights and
+    by sigmoid of the h-th of H numbers W_g x), tensor_names.  Tensors: q, k, v, o, and `sink` [H], `g` [H, hidden], `rel`
+    [rows, H] where asked for; no biases.  With a convolution the caches are (pages, the convolution's inputs); it and the
+    norm run in the launch that writes the cache when every entry brings one token.  q, k, v and the gates are one product of the input; scores, softmax weights and
     their product with the values are fp32 in both engines (the kernels `PlainAttend` picks).  Beside another mixer
     (`parallel_mixers`) it takes the joint product's columns as `proj`, and with a gate a head an `out_scale` on what
     its output product reads and an `add_to` that product is added into."""
@@ -392,6 +410,12 @@ class DistanceBiasAttention(Mixer):
         self.hd, self.vd = int(p["head_dim"]), int(p.get("value_dim") or p["head_dim"])
         self.scale = float(p["scale"])
         self.window = int(p["window"]) if p.get("window") else None
+        self.block = int(p["block"]) if p.get("block") else None
+        self.bias = str(p.get("bias", "slopes"))
+        if self.bias not in ("slopes", "buckets"):
+            raise ValueError(f"distance bias {self.bias!r}: known are 'slopes' and 'buckets'")
+        self.bias_far = float(p["bias_far"]) if self.bias == "buckets" else 0.0
+        self.qk_norm_eps = float(p["qk_norm_eps"]) if p.get("qk_norm_eps") is not None else None
         self.slope_exponent = float(p.get("slope_exponent", 8.0))
         self.sink, self.head_gate = bool(p.get("sink", False)), bool(p.get("head_gate", False))
         self.tensor_names = dict(p.get("tensor_names") or {})
@@ -400,6 +424,9 @@ class DistanceBiasAttention(Mixer):
         if not (1 <= self.hd <= 512 and 1 <= self.vd <= 512):
             raise ValueError(f"head sizes {self.hd}, {self.vd}: the attention kernel takes sizes up to 512")
         self.nq, self.nk, self.nv = self.H * self.hd, self.G * self.hd, self.G * self.vd
+        self.conv = ConvState(self.nq + self.nk + self.nv, int(p["conv_taps"])) if p.get("conv_taps") else None
+        # (beside another mixer the convolution's state would come between the sides' caches)
+        self.joins_input = self.conv is None
         self.scales_output = self.head_gate          # the gate's kernel is where a factor on the output is free
 
     def _name(self, local: str) -> str:
@@ -413,14 +440,26 @@ class DistanceBiasAttention(Mixer):
             d[n("sink")] = ParamDecl((self.H,), init="zeros")
         if self.head_gate:
             d[n("g")] = ParamDecl((self.H, self.hidden))
+        if self.bias == "buckets":
+            d[n("rel")] = ParamDecl((-1, self.H))
+        if self.qk_norm_eps is not None:
+            d[n("q.norm")] = ParamDecl((self.nq,), init="ones")
+            d[n("k.norm")] = ParamDecl((self.nk,), init="ones")
+        if self.conv is not None:
+            for x, size in (("q", self.nq), ("k", self.nk), ("v", self.nv)):
+                d[n(x + ".conv")] = ParamDecl((size, self.conv.taps))
         return d
 
     def cache_need(self):
-        return PagedKV(self.G, self.hd, self.window, value_dim=self.vd if self.vd != self.hd else None)
+        pages = PagedKV(self.G, self.hd, self.window, value_dim=self.vd if self.vd != self.hd else None, block=self.block)
+        return pages if self.conv is None else (pages, self.conv.need())
 
     def prepare(self, ctx: BuildContext) -> None:
         super().prepare(ctx)
-        self.attend = PlainAttend(ctx, self.H, self.G, self.hd, self.vd, window=self.window)
+        self.attend = PlainAttend(ctx, self.H, self.G, self.hd, self.vd, window=self.window, block=self.block)
+        self.slopes = None
+        if self.bias != "slopes":
+            return
         slopes = [2.0 ** (-self.slope_exponent * (h + 1) / self.H) for h in range(self.H)]
         self.slopes = torch.tensor(slopes, dtype=torch.float64).to(torch.float32).to(ctx.device)
 
@@ -434,26 +473,46 @@ class DistanceBiasAttention(Mixer):
         self.proj = Linear(torch.cat([t.to(dt) for t in parts], dim=0), self.ctx.num_sms)
         self.o = Linear(tensors[n("o")], self.ctx.num_sms)
         self.sink_values = tensors[n("sink")].to(torch.float32).contiguous() if self.sink else None
+        self.bias_rows = self.q_norm = self.k_norm = None
+        if self.bias == "buckets":
+            reach = min([r for r in (self.window, self.block) if r], default=None)
+            self.bias_rows = bucket_bias(tensors[n("rel")], self.bias_far, reach)
+        if self.qk_norm_eps is not None:
+            self.q_norm, self.k_norm = tensors[n("q.norm")].contiguous(), tensors[n("k.norm")].contiguous()
+        if self.conv is not None:
+            self.conv.load(torch.cat([tensors[n(x + ".conv")] for x in ("q", "k", "v")], dim=0))
 
-    def forward(self, x: torch.Tensor, step: StepContext, cache: PagedLayerCache, proj: Optional[torch.Tensor] = None,
+    def forward(self, x: torch.Tensor, step: StepContext, cache, proj: Optional[torch.Tensor] = None,
                 out_scale: float = 1.0, add_to: Optional[torch.Tensor] = None) -> torch.Tensor:
         T, dt = x.shape[0], self.ctx.dtype
+        conv_cache = None
+        if self.conv is not None:
+            cache, conv_cache = cache
         g = step.groups[cache.group]
         if proj is None:
             proj = self.proj(x, out_dtype=torch.float32)
         nqkv = self.nq + self.nk + self.nv
         q = torch.empty((T, self.nq), dtype=dt, device=x.device)
-        K.qkv_prepare(proj[:, :nqkv], None, None, None, 0, 0.0, step.positions, None, None, 0, False,
-                      g.slot_of_token if cache.writes else None, cache.kv if cache.writes else None, q,
-                      self.H, self.G, self.hd, self.vd, True)
+        qkv, conv = proj[:, :nqkv], None
+        if conv_cache is not None:
+            if step.max_q_len == 1 and step.num_entries == T:
+                conv = (self.conv.weight, conv_cache.state, step.state_slots)
+            else:
+                qkv = self.conv.run(qkv, step, conv_cache, torch.empty((T, nqkv), dtype=torch.float32, device=x.device),
+                                    residual=False)
+        K.qkv_prepare(qkv, None, self.q_norm, self.k_norm, 0 if self.qk_norm_eps is None else 2, self.qk_norm_eps or 0.0,
+                      step.positions, None, None, 0, False, g.slot_of_token if cache.writes else None,
+                      cache.kv if cache.writes else None, q, self.H, self.G, self.hd, self.vd, True, conv=conv)
         if self.head_gate:
             o = torch.empty((T, self.H * self.vd), dtype=torch.float32, device=x.device)
-            self.attend(q, o, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes)
+            self.attend(q, o, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes,
+                        bias=self.bias_rows)
             y = torch.empty((T, self.H * self.vd), dtype=dt, device=x.device)
             K.sigmoid_gate(o, proj[:, nqkv:], self.vd, y, scale=out_scale)
         else:
             if out_scale != 1.0:
                 raise ValueError("a factor on the output rides on the heads' gate; this mixer has none")
             y = torch.empty((T, self.H * self.vd), dtype=dt, device=x.device)
-            self.attend(q, y, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes)
+            self.attend(q, y, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes,
+                        bias=self.bias_rows)
         return project_out(self.o, y, add_to)

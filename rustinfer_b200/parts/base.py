@@ -242,6 +242,18 @@ class PositionEncoding(Part):
     pass
 
 
+def shared_position(ctx: BuildContext, spec: Optional[PartSpec]) -> Optional[Any]:
+    """The position encoding of `spec`, built once for the layers that share it (None: none)."""
+    if spec is None:
+        return None
+    key = ("position", spec.key(), ctx.max_model_len)
+    if key not in ctx.shared:
+        part = POSITIONS.build(spec)
+        part.prepare(ctx)
+        ctx.shared[key] = part
+    return ctx.shared[key]
+
+
 class Embedding(Part):
     """The stem: turns the step's token ids (and, if it wants, positions) into the fp32 stream."""
 

@@ -121,6 +121,39 @@ def _hyper(block: Block, hidden: Hidden, step: StepContext, cache) -> None:
         hidden.pending = HyperPending(block.ffn.forward(x, step), block.ffn_norm)
 
 
+def _stream_rounded(hidden: Hidden, dtype: torch.dtype) -> torch.Tensor:
+    """The stream in the activation dtype: what the block before left in `hidden.act`, or the stem's output rounded."""
+    from ..ops import kernels as K
+    if hidden.pending is not None:
+        raise ValueError("sublayers that read the stream itself follow blocks that leave nothing pending")
+    if hidden.act is not None:
+        return hidden.act
+    if dtype == torch.float32:
+        return hidden.stream
+    x = torch.empty(hidden.stream.shape, dtype=dtype, device=hidden.stream.device)
+    K.round_rows(hidden.stream, x)
+    return x
+
+
+def _output_norm(block: Block, hidden: Hidden, step: StepContext, cache) -> None:
+    """Norms on the sublayers' outputs only:
+
+        h <- h + post_mixer_norm(mixer(h));  h <- h + post_ffn_norm(ffn(h))
+
+    (the second line only when the layer has a feed-forward).  The sublayers read the stream itself, rounded to the
+    activation dtype; the norms (`rmsnorm` parts) add into the fp32 stream and hand out its rounding for the next sublayer in
+    the same launch.  A feed-forward of experts leaves its weighted sum to that launch too."""
+    post_mixer, post_ffn = block.extra_norms.get("post_mixer_norm"), block.extra_norms.get("post_ffn_norm")
+    if post_mixer is None or (block.ffn is not None and post_ffn is None):
+        raise ValueError("the output_norm arrangement wants a norm after each sublayer")
+    x = _stream_rounded(hidden, post_mixer.ctx.dtype)
+    x = post_mixer.add_output(hidden.stream, block.mixer.forward(x, step, cache))
+    if block.ffn is not None:
+        rows = getattr(block.ffn, "forward_rows", None)
+        x = post_ffn.add_output(hidden.stream, rows(x, step) if rows is not None else block.ffn.forward(x, step))
+    hidden.act = x
+
+
 def _post_norm(block: Block, hidden: Hidden, step: StepContext, cache) -> None:
     """The norm after the sum, and the stream replaced by it:
 
@@ -130,18 +163,10 @@ def _post_norm(block: Block, hidden: Hidden, step: StepContext, cache) -> None:
     both norms are `post_rmsnorm` parts, which hold alpha.  The stream is fp32; each norm also hands
     out its result rounded to the activation dtype, which is what the next sublayer's products read
     (`hidden.act`; the first block of a model rounds the stem's output itself)."""
-    from ..ops import kernels as K
     from .norm import PostRMSNorm
     if not isinstance(block.mixer_norm, PostRMSNorm) or (block.ffn is not None and not isinstance(block.ffn_norm, PostRMSNorm)):
         raise ValueError("the post_norm arrangement wants a post_rmsnorm after each sublayer")
-    if hidden.pending is not None:
-        raise ValueError("the post_norm arrangement follows blocks that leave nothing pending")
-    x = hidden.act
-    if x is None:
-        x = hidden.stream
-        if block.mixer_norm.ctx.dtype != torch.float32:
-            x = torch.empty(hidden.stream.shape, dtype=block.mixer_norm.ctx.dtype, device=hidden.stream.device)
-            K.round_rows(hidden.stream, x)
+    x = _stream_rounded(hidden, block.mixer_norm.ctx.dtype)
     x = block.mixer_norm.renorm(hidden.stream, block.mixer.forward(x, step, cache))
     if block.ffn is not None:
         x = block.ffn_norm.renorm(hidden.stream, block.ffn.forward(x, step))
@@ -235,7 +260,7 @@ def _sandwich_depth_average(block: Block, hidden: Hidden, step: StepContext, cac
 
 
 ARRANGEMENTS: Dict[str, Callable] = {"pre_norm": _pre_norm, "sandwich": _sandwich, "hyper": _hyper,
-                                     "post_norm": _post_norm, "sandwich_depth_average": _sandwich_depth_average}
+                                     "post_norm": _post_norm, "output_norm": _output_norm, "sandwich_depth_average": _sandwich_depth_average}
 
 
 def register_arrangement(name: str, fn: Callable) -> None:

@@ -7,6 +7,8 @@ chosen by a router, and through a shared one where the model has it.
     the `top` largest c are chosen; their weights are the s (divided by their sum when `renormalize`)
     y = sum_chosen weight_e * down_e( silu(gate_e x) * up_e x ) + shared(x)
 
+With `score` "softmax" the scores s are the softmax of z over all experts; with `group_score` "max" a group's score is
+its largest c; `shared_gate`: the shared expert's row is multiplied by sigmoid(w_sg . x), one number a token.
 With `score` "softmax_chosen" the `top` largest logits z are chosen as they are and the weights are their softmax
 among themselves.  With `activation` "clamped" an expert is down_e( g' sigmoid(alpha g') (u' + 1) ) with
 g' = min(gate_e x, limit) and u' = clamp(up_e x, -limit, limit).
@@ -19,7 +21,8 @@ captured in a step's CUDA graph.  The reference engine has dense feed-forwards o
 from __future__ import annotations
 
 import os
-from typing import Dict, Optional
+from dataclasses import dataclass
+from typing import Dict, Optional, Tuple
 
 import torch
 
@@ -28,12 +31,20 @@ from .base import FEED_FORWARDS, FeedForward, ParamDecl, StepContext, register_f
 from .spec import PartSpec
 
 
+@dataclass
+class ExpertRows:
+    """What a feed-forward of experts leaves when its weighted sum is the next kernel's work: the arguments of
+    `kernels.moe_combine` (rows in expert order, places, weights, shared rows, their factor, the counters)."""
+    args: Tuple
+
+
 @register_feed_forward("routed_experts")
 class RoutedExperts(FeedForward):
     """params: hidden_size, expert_ff, experts, top, groups_count / groups_keep (None: no groups), shared_ff
-    (None: no shared expert), score ("sigmoid", or "softmax_chosen"), activation ("silu", or "clamped" with
+    (None: no shared expert), score ("sigmoid", "softmax" or "softmax_chosen"), group_score ("top2", the sum of a
+    group's two largest, or "max"), shared_gate (a tensor `sg` [1, hidden] beside the shared expert's), activation ("silu", or "clamped" with
     `limit` and `alpha`, default 1.702), correction (the router has a tensor added to the scores for
-    the choice), renormalize, output ("float32", the default, or the activation dtype); tensor names:
+    the choice), renormalize (with renormalize_eps added to the sum, default 0), output ("float32", the default, or the activation dtype); tensor names:
     expert_prefix (default "e{}."; `{}` is the expert's number), gate_name / up_name / down_name (default
     "gate" / "up" / "down"), router_name ("router"), correction_name ("correction"), shared_prefix ("shared.")."""
 
@@ -48,8 +59,15 @@ class RoutedExperts(FeedForward):
         self.keep = int(p["groups_keep"]) if p.get("groups_keep") else 0
         self.shared_ff = int(p["shared_ff"]) if p.get("shared_ff") else None
         self.score = str(p.get("score", "sigmoid"))
-        if self.score not in ("sigmoid", "softmax_chosen"):
-            raise ValueError(f"router score {self.score!r}: known are 'sigmoid' and 'softmax_chosen'")
+        if self.score not in ("sigmoid", "softmax", "softmax_chosen"):
+            raise ValueError(f"router score {self.score!r}: known are 'sigmoid', 'softmax' and 'softmax_chosen'")
+        self.group_score = str(p.get("group_score", "top2"))
+        if self.group_score not in ("top2", "max"):
+            raise ValueError(f"group score {self.group_score!r}: known are 'top2' and 'max'")
+        self.renorm_eps = float(p.get("renormalize_eps", 0.0))
+        self.shared_gate = bool(p.get("shared_gate", False))
+        if self.shared_gate and not self.shared_ff:
+            raise ValueError("a gate of the shared expert goes with a shared expert")
         activation = str(p.get("activation", "silu"))
         if activation not in ("silu", "clamped"):
             raise ValueError(f"expert activation {activation!r}: known are 'silu' and 'clamped'")
@@ -93,6 +111,8 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             for local, decl in self.shared.param_decls().items():
                 d[self.shared_prefix + self._shared_names[local]] = decl
+        if self.shared_gate:
+            d[self.shared_prefix + "sg"] = ParamDecl((1, self.hidden))
         return d
 
     def prepare(self, ctx) -> None:
@@ -110,6 +130,9 @@ class RoutedExperts(FeedForward):
         self.down = torch.stack([tensors[p + n["down"]] for p in pre]).contiguous()
         # the router is 32-bit in both engines; the choice kernel forms its product itself
         self.router = tensors[n["router"]].to(torch.float32).contiguous()
+        if self.shared_gate:                                 # one row more: its product's sigmoid is the shared expert's factor
+            sg = tensors[self.shared_prefix + "sg"].to(torch.float32)
+            self.router = torch.cat([self.router, sg], dim=0).contiguous()
         self.correction = tensors[n["correction"]].to(torch.float32).contiguous() if self.has_correction else None
         self.counts = torch.zeros(self.E, dtype=torch.int32, device=self.gate_up.device)   # the kernels leave it zero
         self.tensor_memory = (self.gate_up.dtype == torch.bfloat16 and self.gate_up.is_cuda
@@ -120,18 +143,31 @@ class RoutedExperts(FeedForward):
             self.shared.load({local: tensors[self.shared_prefix + name] for local, name in self._shared_names.items()})
 
     def route(self, x: torch.Tensor):
-        """(ids int32 [T, top], weights fp32 [T, top]); adds the choices to `self.counts`."""
+        """(ids int32 [T, top], weights fp32 [T, top], the shared expert's factor fp32 [T] or None); adds the choices to
+        `self.counts`."""
         T = x.shape[0]
         ids = torch.empty((T, self.top), dtype=torch.int32, device=x.device)
         weights = torch.empty((T, self.top), dtype=torch.float32, device=x.device)
+        gate = torch.empty(T, dtype=torch.float32, device=x.device) if self.shared_gate else None
         K.moe_route(None, self.correction, self.top, self.groups, self.keep, self.renorm, ids, weights, self.counts,
-                    x=x if x.is_contiguous() else x.contiguous(), router=self.router, score=self.score)
-        return ids, weights
+                    x=x if x.is_contiguous() else x.contiguous(), router=self.router, score=self.score,
+                    group_score=self.group_score, renorm_eps=self.renorm_eps, gate=gate)
+        return ids, weights, gate
+
+    def forward_rows(self, x: torch.Tensor, step: StepContext) -> ExpertRows:
+        """Everything but the weighted sum of a token's rows, for a norm that forms it in its own launch."""
+        return ExpertRows(self._rows(x, step))
 
     def forward(self, x: torch.Tensor, step: StepContext, residual: Optional[torch.Tensor] = None):
+        Y, place, weights, shared, gate, counts = self._rows(x, step)
+        out = torch.empty((x.shape[0], self.hidden), dtype=torch.float32 if self.out_fp32 else self.ctx.dtype, device=x.device)
+        K.moe_combine(Y, place, weights, shared, out, counts, gate)
+        return out
+
+    def _rows(self, x: torch.Tensor, step: StepContext) -> Tuple:
         T, dev = x.shape[0], x.device
         N = T * self.top
-        ids, weights = self.route(x)
+        ids, weights, gate = self.route(x)
         offsets = torch.empty(self.E + 1, dtype=torch.int32, device=dev)
         order = torch.empty(N, dtype=torch.int32, device=dev)
         place = torch.empty(N, dtype=torch.int32, device=dev)
@@ -151,6 +187,4 @@ class RoutedExperts(FeedForward):
             K.moe_product(xin, self.gate_up, mid, offsets, order, self.top, gated=True, act=self.act)
             K.moe_product(mid, self.down, Y, offsets, None, self.top, gated=False)
         shared = self.shared.forward(x, step) if self.shared is not None else None
-        out = torch.empty((T, self.hidden), dtype=torch.float32 if self.out_fp32 else self.ctx.dtype, device=dev)
-        K.moe_combine(Y, place, weights, shared, out, self.counts)
-        return out
+        return Y, place, weights, shared, gate, self.counts

@@ -67,11 +67,11 @@ class Linear:
         K.gemm_tc(x, self.weight, out, K.EPI_RELU2, num_sms=self.num_sms)
         return out
 
-    def silu_pairs(self, x: torch.Tensor) -> Optional[torch.Tensor]:
-        """For a weight whose rows alternate gate_j, up_j: silu(gate) * up, [M, out/2], fused
-        into the product's epilogue; None if this weight cannot take that path."""
+    def gated_pairs(self, x: torch.Tensor, gelu: bool = False) -> Optional[torch.Tensor]:
+        """For a weight whose rows alternate gate_j, up_j: silu(gate) * up (with `gelu` gelu_tanh(gate) * up),
+        [M, out/2], fused into the product's epilogue; None if this weight cannot take that path."""
         if not self._own(x) or self.out_features % 2:
             return None
         out = torch.empty((x.shape[0], self.out_features // 2), dtype=torch.bfloat16, device=x.device)
-        K.gemm_tc(x, self.weight, out, K.EPI_SILU, num_sms=self.num_sms)
+        K.gemm_tc(x, self.weight, out, K.EPI_GELU if gelu else K.EPI_SILU, num_sms=self.num_sms)
         return out

@@ -9,6 +9,8 @@ prompt, a portion of one and a single decoded token are the same kernel launch.
     delta_rule               S_t = diag(w_t) S_{t-1} - (a_t * u_t)(u_t^T S_{t-1}) + k_t v_t^T,  o_t = S_t^T r_t
                              u = k / sqrt(|k|^2 + unit_eps),  w = exp(-decay_rate * sigmoid(W_w2 tanh(W_w1 h) + w0)),
                              a = sigmoid(W_a h + b);  out = W_o( rms_head(o) * w * sigmoid(W_g h) )
+    lightning_attention      one fixed decay a head, activated inputs, a norm over all heads with a gate
+    retention                one fixed decay a head, rotated keys and queries, a norm a head with a gate
 
 The projections of one input are one matrix product (rows of the weights joined); the low-rank
 pair that makes the decay is two small products, the second with fp32 output.  Decays, gates of
@@ -25,7 +27,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..ops import kernels as K
-from .base import FixedState, Mixer, ParamDecl, StateLayerCache, StepContext, register_mixer
+from .base import FixedState, Mixer, ParamDecl, StateLayerCache, StepContext, register_mixer, shared_position
 from .linear import Linear
 
 
@@ -243,4 +245,78 @@ class LightningAttention(Mixer):
                      cache.state, step.cu_q, step.state_slots, step.num_entries, self.H, self.dk, self.dv)
         y = torch.empty((T, vg), dtype=self.ctx.dtype, device=x.device)
         K.row_norm_gate(o, p[:, 2 * qk + vg:], self.norm_w, self.norm_eps, y)
+        return self.o(y, out_dtype=torch.float32)
+
+
+@register_mixer("retention")
+class Retention(Mixer):
+    """Linear attention with one fixed decay a head and rotated queries and keys (Sun et al., "Retentive Network: A
+    Successor to Transformer for Large Language Models"):
+
+        q = rot(W_q h), k = rot(W_k h) * k_scale, v = W_v h;  S_t = decay_h S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t
+        out = W_o( rms_head(o) * silu(W_g h) )
+
+    params: hidden_size, num_heads, key_dim, value_dim, decay (one number per head), k_scale (default key_dim^(-1/2)),
+    position (PartSpec of a rotary encoding over key_dim, or None), norm_eps, tensor_names.  Tensors: q, k [H*dk, hidden]; v, g
+    [H*dv, hidden]; o [hidden, H*dv].  The four projections are one product whose result stays fp32; rotation, decays, the
+    state, the norm and the gate are fp32 in both engines.  k_scale is multiplied into the queries instead (the state then
+    holds unscaled keys).  Steps of single tokens rotate in the launch of the recurrence's step."""
+    graph_safe = True
+    joined = ["q", "k", "v", "g"]
+
+    def __init__(self, params):
+        super().__init__(params)
+        p = params
+        self.hidden = int(p["hidden_size"])
+        self.H, self.dk = int(p["num_heads"]), int(p["key_dim"])
+        self.dv = int(p.get("value_dim") or self.dk)
+        self.decay = [float(x) for x in p["decay"]]
+        self.k_scale = float(p["k_scale"]) if p.get("k_scale") is not None else self.dk ** -0.5
+        self.norm_eps = float(p["norm_eps"])
+        self.position_spec = p.get("position")
+        self.tensor_names = dict(p.get("tensor_names") or {})
+        if len(self.decay) != self.H:
+            raise ValueError(f"{len(self.decay)} decays for {self.H} heads")
+        if not (1 <= self.dk <= 512 and self.dv >= 1):
+            raise ValueError(f"key size {self.dk}: the recurrence kernels take key sizes up to 512")
+
+    def _name(self, local: str) -> str:
+        return self.tensor_names.get(local, local)
+
+    def param_decls(self) -> Dict[str, ParamDecl]:
+        n, qk, vg = self._name, self.H * self.dk, self.H * self.dv
+        return {n("q"): ParamDecl((qk, self.hidden)), n("k"): ParamDecl((qk, self.hidden)),
+                n("v"): ParamDecl((vg, self.hidden)), n("g"): ParamDecl((vg, self.hidden)),
+                n("o"): ParamDecl((self.hidden, vg))}
+
+    def cache_need(self):
+        return FixedState((self.H, self.dv, K.recurrent_state_rows(self.dk)), "float32")
+
+    def prepare(self, ctx) -> None:
+        super().prepare(ctx)
+        self.decay_row = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(ctx.device)
+        self.position = shared_position(ctx, self.position_spec)
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        n = self._name
+        parts = [tensors[n(x)] for x in self.joined]
+        dt = torch.float32 if any(t.dtype == torch.float32 for t in parts) else parts[0].dtype
+        self.proj = Linear(torch.cat([t.to(dt) for t in parts], dim=0), self.ctx.num_sms)
+        self.o = Linear(tensors[n("o")], self.ctx.num_sms)
+
+    def forward(self, x: torch.Tensor, step: StepContext, cache: StateLayerCache) -> torch.Tensor:
+        T, qk, vg = x.shape[0], self.H * self.dk, self.H * self.dv
+        p = self.proj(x, out_dtype=torch.float32)
+        pos, rotation = self.position, None
+        if pos is not None:
+            inter = pos.layout == "interleaved"
+            if T == step.num_entries:                            # single tokens: rotated on their way into the recurrence
+                rotation = (step.positions, pos.cos, pos.sin, pos.rotary_dim, inter)
+            else:
+                K.rotate_cols(p[:, : 2 * qk], step.positions, pos.cos, pos.sin, 2 * self.H, self.dk, pos.rotary_dim, inter)
+        o = torch.empty((T, vg), dtype=torch.float32, device=x.device)
+        K.head_scan(p[:, :qk], p[:, qk: 2 * qk], p[:, 2 * qk: 2 * qk + vg], self.decay_row, self.k_scale, o, cache.state,
+                    step.cu_q, step.state_slots, step.num_entries, self.H, self.dk, self.dv, rotation=rotation)
+        y = torch.empty((T, vg), dtype=self.ctx.dtype, device=x.device)
+        K.part_norm_gate(o, p[:, 2 * qk + vg:], None, self.H, self.norm_eps, False, y)
         return self.o(y, out_dtype=torch.float32)

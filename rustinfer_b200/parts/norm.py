@@ -17,8 +17,8 @@ from .base import Norm, ParamDecl, register_norm
 class RMSNorm(Norm):
     """params: size, eps, weight_name (the tensor's local name, default "weight"), offset (added to the stored
     weight: 1 for a weight stored around zero; default 0), scale (a factor on the norm's output, the residual's
-    factor of a norm that follows a sublayer, say; default 1).  With an offset or a scale the part keeps
-    (offset + w) * scale in fp32.
+    factor of a norm that follows a sublayer, say; default 1), scalar (True: the stored weight is one number, shape [],
+    for all channels).  With an offset, a scale or one number the part keeps (offset + w) * scale in fp32.
 
     `add_norm` takes as `delta` a tensor (added as it is), None, a `NormedDelta` (normed by the RMS norm it names,
     then added) or a `DepthPending` (see parts/block.py); the last two run as one kernel with this norm."""
@@ -30,15 +30,21 @@ class RMSNorm(Norm):
         self.weight_name = str(params.get("weight_name", "weight"))
         self.offset = float(params.get("offset", 0.0))
         self.scale = float(params.get("scale", 1.0))
+        self.scalar = bool(params.get("scalar", False))
         self.weight: Optional[torch.Tensor] = None
         self._weight32: Optional[torch.Tensor] = None
 
     def param_decls(self) -> Dict[str, ParamDecl]:
-        return {self.weight_name: ParamDecl((self.size,), init="zeros" if self.offset == 1.0 else "ones")}
+        return {self.weight_name: ParamDecl(() if self.scalar else (self.size,), init="zeros" if self.offset == 1.0 else "ones")}
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         w = tensors[self.weight_name].contiguous()
-        if self.offset != 0.0 or self.scale != 1.0:
+        self._one = None
+        if self.scalar:
+            # the kernel that norms a sublayer's output reads the one number; the others a row of it
+            self._one = ((w.to(torch.float32) + self.offset) * self.scale).reshape(1).contiguous()
+            w = self._one.expand(self.size).contiguous()
+        elif self.offset != 0.0 or self.scale != 1.0:
             w = ((w.to(torch.float32) + self.offset) * self.scale).contiguous()
         self.weight = w
         self._weight32 = None
@@ -78,6 +84,18 @@ class RMSNorm(Norm):
             return out
         K.add_rmsnorm(h, delta, self.weight, self.eps, out, rows)
         return out
+
+    def add_output(self, h: torch.Tensor, y) -> torch.Tensor:
+        """h <- h + rms(y) * w in place, y a sublayer's output (or `ExpertRows`, whose sum the same launch forms); returns
+        the new h in the activation dtype for the next sublayer (h itself in a 32-bit engine)."""
+        from .experts import ExpertRows
+        act = None if self.ctx.dtype == torch.float32 else torch.empty(h.shape, dtype=self.ctx.dtype, device=h.device)
+        w = self._one if self.scalar else self.weight32
+        if isinstance(y, ExpertRows):
+            K.norm_add(h, None, w, self.eps, act, experts=y.args)
+        else:
+            K.norm_add(h, y, w, self.eps, act)
+        return h if act is None else act
 
     def add_into(self, h: torch.Tensor, delta: torch.Tensor, h_out: Optional[torch.Tensor] = None) -> None:
         """h_out (default h itself) <- h + rms(delta) * w."""

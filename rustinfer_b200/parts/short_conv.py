@@ -6,7 +6,8 @@
 fixed-state cache group of the part's own), so a prompt cut into portions and a token decoded alone see the same
 inputs as the whole prompt would.  The convolution runs in fp32 on the fp32 output of the norm before it and is
 rounded once, for the mixer's products.  `ConvState` is the same convolution for mixers that have one inside
-(the recurrent unit's input branch).  The reference engine has no such part (its blocks are
+(the recurrent unit's input branch; an attention's q, k and v; a state-space mixer's inputs, with its activation and the
+step sizes that lie behind its channels).  The reference engine has no such part (its blocks are
 crates/infer-worker/src/components/decoder_block.rs:13-32).
 """
 from __future__ import annotations
@@ -22,8 +23,11 @@ from .base import MIXERS, BuildContext, FixedState, Mixer, ParamDecl, StateLayer
 class ConvState:
     """The convolution's weights ([channels, taps], kept fp32) and how it is run on a step."""
 
-    def __init__(self, channels: int, taps: int):
+    def __init__(self, channels: int, taps: int, activation: Optional[str] = None):
         self.channels, self.taps = int(channels), int(taps)
+        if activation not in (None, "silu"):
+            raise ValueError(f"a short convolution's activation: known is 'silu', got {activation!r}")
+        self.silu = activation == "silu"
         if not 1 <= self.taps <= 8:
             raise ValueError(f"a short convolution has 1 to 8 taps, got {self.taps}")
         self.weight: Optional[torch.Tensor] = None
@@ -37,9 +41,9 @@ class ConvState:
         self.bias = bias.to(torch.float32).contiguous() if bias is not None else None
 
     def run(self, x: torch.Tensor, step: StepContext, cache: StateLayerCache, out: torch.Tensor, residual: bool,
-            in_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+            in_bias: Optional[torch.Tensor] = None, steps=None) -> torch.Tensor:
         K.short_conv(x, self.weight, self.bias, cache.state, step.cu_q, step.state_slots, out, step.num_entries,
-                     step.max_q_len, residual, in_bias)
+                     step.max_q_len, residual, in_bias, self.silu, steps)
         return out
 
 
