@@ -110,7 +110,8 @@ __device__ __forceinline__ void load_tile(bf16* Ks, bf16* Vs, const bf16* __rest
     }
 }
 
-template <typename TO, bool VIK>
+// BIAS: the scores carry the learned distance bias (an instantiation of its own: it costs registers)
+template <typename TO, bool VIK, bool BIAS>
 __global__ void __launch_bounds__(THREADS, VD <= 128 ? (VIK ? 4 : 3) : 1)      // values to 128 wide: three or four CTAs an SM
 attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__ out, int out_stride,
                       const bf16* __restrict__ cache, const int* __restrict__ block_table, int table_stride,
@@ -174,14 +175,14 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
     int p_row[2], lo_row[2];
     bool ok_row[2];
     float m[2], l[2] = {0.f, 0.f}, slope[2] = {0.f, 0.f};
-    const float* bias[2] = {nullptr, nullptr};
+    int bias_row[2] = {0, 0};
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         const int r = warp * 16 + (lane >> 2) + 8 * i;
         const int jj = r / Gc, hh = r - jj * Gc;
         ok_row[i] = jj < ntok && hh < nheads;
         if (gm.slopes && ok_row[i]) slope[i] = gm.slopes[head_of(hh)];
-        if (gm.bias) bias[i] = gm.bias + (size_t)(ok_row[i] ? head_of(hh) : 0) * gm.bias_len;
+        if (BIAS && ok_row[i]) bias_row[i] = head_of(hh) * gm.bias_len;
         p_row[i] = p_first + jj;
         lo_row[i] = gm.window > 0 ? max(0, p_row[i] - gm.window + 1) : 0;
         if (gm.block > 0) lo_row[i] = max(lo_row[i], p_row[i] / gm.block * gm.block);
@@ -247,7 +248,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
                     float sc = s[n][e] * gm.scale;
                     if (gm.softcap > 0.f) sc = gm.softcap * tanhf(sc / gm.softcap);
                     sc -= slope[i] * (float)(p_row[i] - key);
-                    if (gm.bias) sc += __ldg(bias[i] + max(0, min(p_row[i] - key, gm.bias_len - 1)));
+                    if (BIAS) sc += __ldg(gm.bias + bias_row[i] + max(0, min(p_row[i] - key, gm.bias_len - 1)));
                     const bool seen = ok_row[i] && key <= p_row[i] && key >= lo_row[i];
                     s[n][e] = seen ? sc * LOG2E : -INFINITY;
                     mx[i] = fmaxf(mx[i], s[n][e]);
@@ -414,19 +415,19 @@ attention_rows_merge_kernel(const float* __restrict__ part, TO* __restrict__ out
     }
 }
 
-template <typename TO, bool VIK>
+template <typename TO, bool VIK, bool BIAS>
 int launch(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
            int table_stride, const int* cu_q, const int* kv_len, const int* tile_entry, const int* tile_tok0,
            int n_tiles, const float* sink_values, float* part, const Geometry& gm, cudaStream_t s) {
     static bool configured = false;
     const size_t smem = ((size_t)MT * KROW + 2 * ((size_t)KT * KROW + (VIK ? 0 : (size_t)KT * VROW))) * sizeof(bf16);
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(n_tiles, gm.Hkv * gm.maps * gm.chunks, gm.splits);
-    RI_CHECKED(ri_launch(attention_rows_kernel<TO, VIK>, grid, dim3(THREADS), smem, s, (const bf16*)q, q_stride, (TO*)out,
+    RI_CHECKED(ri_launch(attention_rows_kernel<TO, VIK, BIAS>, grid, dim3(THREADS), smem, s, (const bf16*)q, q_stride, (TO*)out,
                          out_stride, (const bf16*)cache, block_table, table_stride, cu_q, kv_len, tile_entry, tile_tok0,
                          sink_values, part, gm));
     if (gm.splits > 1)
@@ -458,8 +459,8 @@ RI_API int ri_attention_rows_ctas_per_sm(int value_in_key, int out_f32) {
     cudaError_t e = cudaErrorInvalidValue;
 #define RI_ROWS_OCC(TO, VIK) do { \
         const size_t smem = ((size_t)MT * KROW + 2 * ((size_t)KT * KROW + (VIK ? 0 : (size_t)KT * VROW))) * sizeof(bf16); \
-        e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attention_rows_kernel<TO, VIK>, THREADS, smem); \
+        e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attention_rows_kernel<TO, VIK, false>, THREADS, smem); \
     } while (0)
     if (value_in_key) {
         if constexpr (VD <= HD) { if (out_f32) RI_ROWS_OCC(float, true); else RI_ROWS_OCC(bf16, true); }
@@ -490,13 +491,15 @@ RI_API int ri_attention_rows(const void* q, int q_stride, void* out, int out_str
     Geometry gm{Hq, Hkv, maps, gc, (G + gc - 1) / gc, MT / gc, page_size, window, sink, splits, scale, softcap, slopes,
                 bias, bias_len, block};
     cudaStream_t s = (cudaStream_t)stream;
-#define RI_ROWS_GO(TO, VIK) launch<TO, VIK>(q, q_stride, out, out_stride, cache, block_table, table_stride, cu_q, kv_len, \
+    if (bias && value_in_key) return (int)cudaErrorNotSupported;
+#define RI_ROWS_GO(TO, VIK, BIAS) launch<TO, VIK, BIAS>(q, q_stride, out, out_stride, cache, block_table, table_stride, cu_q, kv_len, \
                                             tile_entry, tile_tok0, n_tiles, sink_values, part, gm, s)
     if (value_in_key) {
-        if constexpr (VD <= HD) return out_f32 ? RI_ROWS_GO(float, true) : RI_ROWS_GO(bf16, true);
+        if constexpr (VD <= HD) return out_f32 ? RI_ROWS_GO(float, true, false) : RI_ROWS_GO(bf16, true, false);
         return (int)cudaErrorInvalidValue;
     }
-    return out_f32 ? RI_ROWS_GO(float, false) : RI_ROWS_GO(bf16, false);
+    if (bias) return out_f32 ? RI_ROWS_GO(float, false, true) : RI_ROWS_GO(bf16, false, true);
+    return out_f32 ? RI_ROWS_GO(float, false, false) : RI_ROWS_GO(bf16, false, false);
 #undef RI_ROWS_GO
 }
 

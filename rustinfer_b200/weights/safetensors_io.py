@@ -149,6 +149,6 @@ def write_safetensors(path: str, tensors: Mapping[str, torch.Tensor]) -> None:
         f.write(struct.pack("<Q", len(blob)))
         f.write(blob)
         for name in order:
-            t = tensors[name].detach().cpu().contiguous()
+            t = tensors[name].detach().cpu().contiguous().reshape(-1)          # a single number is a row of one
             f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
     os.replace(tmp, path)
