@@ -17,7 +17,7 @@ attention), the Llama-3.2-3B-shaped model at 8 of its 28 layers serving 64 reque
 this engine's attention and GEMM kernels timed against the reference's own attention kernels
 (compiled unmodified, see baseline/reference_kernels.py) and the library GEMM on the same data.
 `--shape` takes the layer sizes of the 3B or 8B benchmark configuration for the headline instead;
-`--only decode|prefill|serve` runs one part alone and prints its time.  `--family dirurax` (or `pikalix`, `sotazen`, `linedra`) leaves
+`--only decode|prefill|serve` runs one part alone and prints its time.  `--family dirurax` (or `pikalix`, `sotazen`, `linedra`, `dozotar`) leaves
 all of that aside and prints a line of its own: prefill and decode of that family's models at two sizes beside
 Llama models of the same width, depth, feed-forward width and vocabulary, and that family's kernels alone against
 their rooflines.
@@ -1149,8 +1149,216 @@ def linedra_kernels(hbm_gbs, bf16_tflops, size):
     return out
 
 
+def _dozotar(width, layers, ff, vocab, attn, chunk, mamba, retention, experts, top, expert_ff, shared_ff, groups):
+    """`layers` layers in the order state space, attention, retention, state space (norms on the outputs); feed-forwards
+    alternate between a dense one and routed experts with a gated shared one."""
+    ah, akv, ad, av, taps = attn
+    mh, mv, mn, mg, mt, mp = mamba
+    rh, rd, rv = retention
+    out = []
+    for i in range(layers):
+        mlp = {"kind": "dense", "ff": ff} if i % 2 == 0 else {
+            "kind": "moe", "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff},
+            "router": {"experts": experts, "top": top, "groups": {"count": groups[0], "keep": groups[1]}}}
+        if i % 4 == 1:
+            out.append({"type": "attention", "mlp": mlp, "mixer": {
+                "heads": ah, "kv_heads": akv, "dim": ad, "vdim": av, "conv": taps, "scale": ad ** -0.5, "bias_max": chunk // 2,
+                "mask": {"size": chunk}}})
+        elif i % 4 == 2:
+            decay = [1.0 - 2.0 ** (-5.0 - 3.0 * h / max(rh - 1, 1)) for h in range(rh)]
+            out.append({"type": "retention", "mlp": mlp, "mixer": {"heads": rh, "dim": rd, "vdim": rv, "decay": decay,
+                                                                   "rot": {"dims": rd, "base": 10000.0}}})
+        else:
+            out.append({"type": "mamba2", "mlp": mlp, "mixer": {"heads": mh, "vdim": mv, "state": mn, "groups": mg, "conv": mt,
+                                                                "norm_groups": mp}})
+    return {"architecture": "Dozotar", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "layers": out}
+
+
+# Dozotar at the same widths: attention (heads, kv heads, key, value, taps), chunks as wide as the other families' windows,
+# the state-space mixer (heads, value, state, groups, taps, norm parts: 2 x width channels), retention (heads, key, value) as
+# Sotazen's walk with fixed decays, feed-forwards as Pikalix's; both stand beside it at equal size
+DOZOTAR_SIZES = {
+    "w1024": dict(width=1024, layers=8, ff=4096, vocab=32768, attn=(16, 4, 64, 64, 4), chunk=1024, mamba=(32, 64, 128, 4, 4, 4),
+                  retention=(8, 128, 128), experts=32, top=4, expert_ff=768, shared_ff=1024, groups=(8, 4), llama=(16, 4, 64)),
+    "w2048": dict(width=2048, layers=8, ff=8192, vocab=32768, attn=(32, 8, 64, 64, 4), chunk=1024, mamba=(64, 64, 128, 8, 4, 8),
+                  retention=(16, 128, 128), experts=32, top=4, expert_ff=1536, shared_ff=2048, groups=(8, 4), llama=(32, 8, 64)),
+}
+
+
+def dozotar_kernels(hbm_gbs, bf16_tflops, size):
+    """The Dozotar kernels alone at one size, each beside the like kernel of the nearest existing family on the same
+    shapes (the add + RMSNorm of the Llama path and Sotazen's norm after the sum, Sotazen's walk with fixed decays, Linedra's
+    convolution, Sotazen's and Dirurax's norms with a gate, the attention without its bias, Pikalix's router and weighted
+    sum): microseconds, and what that is of the bytes they must move at the measured copy bandwidth."""
+    import torch
+    from rustinfer_b200.ops import kernels as K
+    from rustinfer_b200.parts.attention_variants import PlainAttend, bucket_bias
+    from rustinfer_b200.parts.base import BuildContext
+    dev = torch.device("cuda:0")
+    sz = DOZOTAR_SIZES[size]
+    d = sz["width"]
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    bf = lambda *s: torch.randn(*s, device=dev).to(torch.bfloat16)
+    f32 = lambda *s: torch.randn(*s, device=dev)
+    frac = lambda moved, us: round(moved / (us * 1e-6) / 1e9 / hbm_gbs, 4)
+    timed = lambda fn: time_kernel(fn, flush=flush)
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+    fma_per_s = sms * 128 * 1.9e9
+    out = {}
+
+    def entry(name, us, moved, likes=(), **more):
+        r = {"us": round(us, 1), "hbm_frac": frac(moved, us)}
+        for like, lus, lmoved in likes:
+            r[like + "_us"], r[like + "_hbm_frac"] = round(lus, 1), frac(lmoved, lus)
+        r.update(more)
+        out[name] = r
+    ah, akv, ad, av, at = sz["attn"]
+    mh, mv, mn, mg, mt, mp = sz["mamba"]
+    rh, rd, rv = sz["retention"]
+    E, top, groups = sz["experts"], sz["top"], sz["groups"]
+    for tag, T, entries in (("prefill2048", 2048, 1), ("decode64", 64, 64)):
+        cu = i32([i * (T // entries) for i in range(entries + 1)])
+        slots = i32(list(range(entries)))
+        # the norm of a sublayer's output with the add, one number for weight
+        h, y, one = f32(T, d), f32(T, d), f32(1)
+        xo, d16, w16 = torch.empty(T, d, device=dev, dtype=torch.bfloat16), bf(T, d), bf(d)
+        entry(f"norm_add_{tag}", timed(lambda: K.norm_add(h, y, one, 1e-6, xo)), T * d * (4 + 4 + 4 + 2), [
+            ("add_rmsnorm", timed(lambda: K.add_rmsnorm(h, d16, w16, 1e-6, xo)), T * d * (4 + 4 + 2 + 2)),
+            ("scale_add_norm", timed(lambda: K.scale_add_norm(h, y, None, 1.0, w16, 1e-6, xo)), T * d * (4 + 4 + 4 + 2))])
+        # the same with the weighted sum of the experts formed in it, beside Pikalix's sum alone
+        Y, shared, gate = f32(T * top, d), f32(T, d), torch.rand(T, device=dev)
+        place, wts = torch.randperm(T * top, device=dev).to(torch.int32), torch.rand(T, top, device=dev)
+        counts, ysum = torch.zeros(E, dtype=torch.int32, device=dev), torch.empty(T, d, device=dev)
+        args = (Y, place, wts, shared, gate, counts)
+        entry(f"norm_add_experts_{tag}", timed(lambda: K.norm_add(h, None, one, 1e-6, xo, experts=args)), T * d * (4 * (top + 1) + 4 + 4 + 2), [
+            ("moe_combine", timed(lambda: K.moe_combine(Y, place, wts, shared, ysum, counts)), T * d * (4 * (top + 1) + 4))])
+        # the router
+        x16, router = bf(T, d), f32(E + 1, d)
+        rplain = router[:E].contiguous()
+        ids, rw = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, device=dev)
+        entry(f"router_{tag}", timed(lambda: K.moe_route(None, None, top, *groups, True, ids, rw, counts, x=x16, router=router,
+                                                         score="softmax", group_score="max", renorm_eps=1e-20, gate=gate)),
+              T * d * 2 + (E + 1) * d * 4, [
+            ("sigmoid_router", timed(lambda: K.moe_route(None, None, top, *groups, True, ids, rw, counts, x=x16, router=rplain)),
+             T * d * 2 + E * d * 4)])
+        counts.zero_()
+        # the state-space mixer: convolution with silu and step sizes, the walk, the gated norm
+        I, GN = mh * mv, mg * mn
+        C = I + 2 * GN
+        proj, cw, cb = f32(T, I + C + mh), f32(C, mt), f32(C)
+        dtb, al = f32(mh), f32(mh)
+        cst = torch.zeros(entries + 1, mt - 1, C, device=dev)
+        xbc, sizes = torch.empty(T, C, device=dev), torch.empty(2, T, mh, device=dev)
+        mq = T // entries
+        plain_out = torch.empty(T, C, device=dev)
+        entry(f"conv_silu_steps_{tag}", timed(lambda: K.short_conv(proj[:, I: I + C], cw, cb, cst, cu, slots, xbc, entries, mq, False, silu=True,
+                                                                   steps=(proj[:, I + C:], dtb, al, sizes[0], sizes[1]))),
+              T * C * 8 + 2 * entries * (mt - 1) * C * 4, [
+            ("short_conv", timed(lambda: K.short_conv(proj[:, I: I + C], cw, cb, cst, cu, slots, plain_out, entries, mq, False)),
+             T * C * 8 + 2 * entries * (mt - 1) * C * 4)])
+        ms = torch.zeros(entries + 1, mh, mv, K.recurrent_state_rows(mn), device=dev)
+        yo = torch.empty(T, I, device=dev)
+        us = timed(lambda: K.head_scan(xbc[:, I + GN:], xbc[:, I: I + GN], xbc[:, :I], sizes[1], 1.0, yo, ms, cu, slots, entries, mh, mn, mv,
+                                       gain=sizes[0], key_heads=mg))
+        # Sotazen's walk on the same state: a key head a head and a decay a channel
+        p32 = f32(T, 2 * mh * mn + mh * mv)
+        dec = torch.full((mh * mn,), 0.97, device=dev)
+        us_d = timed(lambda: K.decay_scan(p32[:, :mh * mn], p32[:, mh * mn:2 * mh * mn], p32[:, 2 * mh * mn:], dec, 1.0, yo, ms, cu, slots,
+                                          entries, mh, mn, mv))
+        st = 2 * entries * mh * mn * mv * 4
+        entry(f"state_space_walk_{tag}", us, T * (C + I) * 4 + st,
+              [("decay_scan", us_d, T * (2 * mh * mn + 2 * mh * mv) * 4 + st)],
+              fma_frac=round(2 * T * mh * mn * mv / (us * 1e-6) / fma_per_s, 4),
+              decay_scan_fma_frac=round(2 * T * mh * mn * mv / (us_d * 1e-6) / fma_per_s, 4))
+        del p32
+        nw, D = f32(I), f32(mh)
+        yb = torch.empty(T, I, device=dev, dtype=torch.bfloat16)
+        entry(f"part_norm_gate_{tag}", timed(lambda: K.part_norm_gate(yo, proj[:, :I], nw, mp, 1e-6, True, yb, skip=(D, xbc[:, :I]))),
+              T * I * (4 + 4 + 4 + 2), [
+            ("row_norm_gate", timed(lambda: K.row_norm_gate(yo, proj[:, :I], nw, 1e-6, yb)), T * I * (4 + 4 + 2))])
+        # retention: rotation, walk, the norm a head with its gate
+        qk, vg = rh * rd, rh * rv
+        p = f32(T, 2 * qk + 2 * vg)
+        pos, cos, sin = i32(list(range(T))), f32(T, rd // 2), f32(T, rd // 2)
+        if entries == 1:
+            q16 = bf(T, 2 * qk)
+            entry(f"rotate_cols_{tag}", timed(lambda: K.rotate_cols(p[:, :2 * qk], pos, cos, sin, 2 * rh, rd, rd)), T * 2 * qk * 8, [
+                ("rope_in_place", timed(lambda: K.rope_scatter(q16, pos, cos, sin, None, None, 2 * rh, 0, rd, rd)), T * 2 * qk * 4)])
+        rs = torch.zeros(entries + 1, rh, rv, K.recurrent_state_rows(rd), device=dev)
+        ro, hdec, cdec = torch.empty(T, vg, device=dev), torch.full((rh,), 0.97, device=dev), torch.full((qk,), 0.97, device=dev)
+        rot = (pos, cos, sin, rd, False) if entries == T else None
+        cols = (p[:, :qk], p[:, qk:2 * qk], p[:, 2 * qk:2 * qk + vg])
+        st = 2 * entries * rh * rd * rv * 4
+        us = timed(lambda: K.head_scan(*cols, hdec, 1.0, ro, rs, cu, slots, entries, rh, rd, rv, rotation=rot))
+        us_d = timed(lambda: K.decay_scan(*cols, cdec, 1.0, ro, rs, cu, slots, entries, rh, rd, rv))
+        entry(f"retention_walk_{tag}", us, T * (2 * qk + 2 * vg) * 4 + st, [("decay_scan", us_d, T * (2 * qk + 2 * vg) * 4 + st)],
+              fma_frac=round(2 * T * qk * rv / (us * 1e-6) / fma_per_s, 4))
+        ry, g16, hw = torch.empty(T, vg, device=dev, dtype=torch.bfloat16), bf(T, vg), bf(rv)
+        entry(f"head_norm_gate_{tag}", timed(lambda: K.part_norm_gate(ro, p[:, 2 * qk + vg:], None, rh, 1e-6, False, ry)), T * vg * (4 + 4 + 2), [
+            ("gated_head_norm", timed(lambda: K.gated_head_norm(ro, g16, hw, False, K.GATE_SILU, 1e-6, ry, rh, rv)), T * vg * (4 + 2 + 2))])
+        # q, k, v: convolution, the norm over all heads, the cache write (one launch for single tokens, two for prompts)
+        qc = ah * ad + akv * (ad + av)
+        qkv, qw, qn, kn = f32(T, qc), f32(qc, at), bf(ah * ad), bf(akv * ad)
+        cache = bf(T // PAGE + 1, 2, akv, PAGE, ad)
+        qo, sl = torch.empty(T, ah * ad, device=dev, dtype=torch.bfloat16), i32(list(range(T)))
+        qst = torch.zeros(entries + 1, at - 1, qc, device=dev)
+        prep = lambda x, conv: K.qkv_prepare(x, None, qn, kn, 2, 1e-6, pos, None, None, 0, False, sl, cache, qo, ah, akv, ad, av, True, conv=conv)
+        us_p = timed(lambda: prep(qkv, None))
+        qtmp = torch.empty(T, qc, device=dev)
+
+        def two():
+            K.short_conv(qkv, qw, None, qst, cu, slots, qtmp, entries, mq, False)
+            prep(qtmp, None)
+        us_two = timed(two)
+        us = timed(lambda: prep(qkv, (qw, qst, slots))) if entries == T else us_two
+        moved = T * qc * (4 + 2) + (2 * entries * (at - 1) * qc * 4 if entries == T else T * qc * 8)
+        entry(f"conv_norm_cache_{tag}", us, moved, [("without_conv", us_p, T * qc * (4 + 2))], two_launches_us=round(us_two, 1))
+    # attention in chunks with the bias beside the same kernels without it
+    B, ctx, chunk = 64, 4096, sz["chunk"]
+    nblk = ctx // PAGE
+    bctx = BuildContext(dev, torch.bfloat16, ctx, PAGE, max_batch_seqs=B, num_sms=sms)
+    kv_len, cu, ent = i32([ctx] * B), i32(list(range(B + 1))), i32(list(range(B)))
+    table = torch.randperm(B * nblk, device=dev).to(torch.int32).view(B, nblk).contiguous()
+    bias = bucket_bias(f32(16, ah), chunk // 2, chunk)
+    att = PlainAttend(bctx, ah, akv, ad, av, block=chunk)
+    cache = bf(B * nblk, 2, akv, PAGE, ad)
+    q, o = bf(B, ah * ad), torch.empty(B, ah * av, device=dev, dtype=torch.bfloat16)
+    ranges = att._splits(B, ctx)
+    run = lambda bi: timed(lambda: K.attention_single(q, o, cache, table, cu, kv_len, ent, ah, akv, ad, ad ** -0.5, None, chunk, av,
+                                                      splits=ranges, part=att.part, bias=bi))
+    moved = B * chunk * akv * (ad + av) * 2
+    entry("bucket_attention_decode64", run(bias), moved, [("no_bias", run(None), moved)], ranges=ranges)
+    T = 2048
+    tbl, cup, kvl = i32([list(range(T // PAGE))]), i32([0, T]), i32([T])
+    pc, qp, op = bf(T // PAGE, 2, akv, PAGE, ad), bf(T, ah * ad), torch.empty(T, ah * av, device=dev, dtype=torch.bfloat16)
+    pairs = sum(p % chunk + 1 for p in range(T))
+    tpt = K.attention_rows_tokens_per_tile(ah, akv, ad, av)
+    tl = list(range(0, T, tpt))
+    te, t0 = i32([0] * len(tl)), i32(tl)
+    res = {}
+    for name, bi in (("us", bias), ("no_bias_us", None)):
+        us = timed(lambda: K.attention_rows(qp, op, pc, tbl, cup, kvl, te, t0, ah, akv, ad, ad ** -0.5, None, av, bias=bi, block=chunk))
+        res[name] = round(us, 1)
+        res[name.replace("us", "useful_tflops")] = round(2 * pairs * ah * (ad + av) / (us * 1e-6) / 1e12, 2)
+    rows = K.mma_tokens_per_tile(ah, akv)
+    tl = list(range(0, T, rows))
+    te, t0 = i32([0] * len(tl)), i32(tl)
+    us = timed(lambda: K.attention_prefill_bf16(qp, op, pc, tbl, cup, kvl, te, t0, ah, akv, ad, ad ** -0.5, None, chunk, precise=True))
+    res["pikalix_kernel_us"] = round(us, 1)
+    out["bucket_attention_prefill2048"] = res
+    # the gelu-gated product beside the silu-gated one
+    xg, wg = bf(2048, d), bf(2 * sz["ff"], d)
+    og = torch.empty(2048, sz["ff"], device=dev, dtype=torch.bfloat16)
+    fl = 2 * 2048 * 2 * sz["ff"] * d
+    us, us_s = timed(lambda: K.gemm_tc(xg, wg, og, K.EPI_GELU)), timed(lambda: K.gemm_tc(xg, wg, og, K.EPI_SILU))
+    out["gelu_gated_product_2048"] = {"us": round(us, 1), "bf16_frac": round(fl / (us * 1e-6) / 1e12 / bf16_tflops, 4),
+                                      "silu_us": round(us_s, 1), "silu_bf16_frac": round(fl / (us_s * 1e-6) / 1e12 / bf16_tflops, 4)}
+    return out
+
+
 def family_bench(args) -> int:
-    """`--family dirurax|pikalix|sotazen|linedra`: prefill and decode throughput of that family's models at a few sizes beside
+    """`--family dirurax|pikalix|sotazen|linedra|dozotar`: prefill and decode throughput of that family's models at a few sizes beside
     Llama models of the same width, depth, feed-forward width and vocabulary (random weights), and the
     family's own kernels alone.  One JSON line."""
     import torch
@@ -1163,7 +1371,7 @@ def family_bench(args) -> int:
     say = lambda msg: print(f"[bench] {msg}", file=sys.stderr, flush=True)
     ctx, tokens = min(args.context, 4096), max(2, min(args.prompt_tokens, 8192))
     family = args.family
-    table = {"pikalix": PIKALIX_SIZES, "sotazen": SOTAZEN_SIZES, "linedra": LINEDRA_SIZES}.get(family, FAMILY_SIZES)
+    table = {"pikalix": PIKALIX_SIZES, "sotazen": SOTAZEN_SIZES, "linedra": LINEDRA_SIZES, "dozotar": DOZOTAR_SIZES}.get(family, FAMILY_SIZES)
     result = {"family": family, "dtype": "bf16", "data": "synthetic", "peaks": peak_kind, "points": {}, "kernels": {}}
     sizes = [s for s in table if not args.size or s in args.size.split(",")]
     for size in sizes:
@@ -1174,11 +1382,15 @@ def family_bench(args) -> int:
             own = _sotazen(**{k: v for k, v in sz.items() if k != "llama"})
         elif family == "linedra":
             own = _linedra(**{k: v for k, v in sz.items() if k != "llama"})
+        elif family == "dozotar":
+            own = _dozotar(**{k: v for k, v in sz.items() if k != "llama"})
         else:
             own = _dirurax(sz["width"], sz["layers"], sz["ff"], sz["vocab"], sz["gla"], sz["attn"], sz["delta"], sz["block"])
         configs = {family: own, "llama": _llama_like(sz["width"], sz["layers"], sz["ff"], sz["vocab"], *sz["llama"])}
-        if family == "linedra":                      # also beside the nearest of the other families, at equal size
+        if family in ("linedra", "dozotar"):         # also beside the nearest of the other families, at equal size
             configs["pikalix"] = _pikalix(**{k: v for k, v in PIKALIX_SIZES[size].items() if k != "llama"})
+        if family == "dozotar":
+            configs["sotazen"] = _sotazen(**{k: v for k, v in SOTAZEN_SIZES[size].items() if k != "llama"})
         point = {}
         for fam, cfg in configs.items():
             with tempfile.TemporaryDirectory(prefix="rustinfer_b200_bench_") as tmp:
@@ -1205,13 +1417,15 @@ def family_bench(args) -> int:
                 torch.cuda.empty_cache()
         point["prefill_ratio"] = round(point[family]["prefill_tokens_per_s"] / point["llama"]["prefill_tokens_per_s"], 3)
         point["decode_ratio"] = round(point[family]["decode_tokens_per_s"] / point["llama"]["decode_tokens_per_s"], 3)
-        if "pikalix" in point and family != "pikalix":
-            point["prefill_ratio_to_pikalix"] = round(point[family]["prefill_tokens_per_s"] / point["pikalix"]["prefill_tokens_per_s"], 3)
-            point["decode_ratio_to_pikalix"] = round(point[family]["decode_tokens_per_s"] / point["pikalix"]["decode_tokens_per_s"], 3)
+        for near in ("pikalix", "sotazen"):
+            if near in point and family != near:
+                point[f"prefill_ratio_to_{near}"] = round(point[family]["prefill_tokens_per_s"] / point[near]["prefill_tokens_per_s"], 3)
+                point[f"decode_ratio_to_{near}"] = round(point[family]["decode_tokens_per_s"] / point[near]["decode_tokens_per_s"], 3)
         result["points"][size] = point
         result["kernels"][size] = (pikalix_kernels(hbm_gbs, bf16_tflops, size) if family == "pikalix"
                                    else sotazen_kernels(hbm_gbs, bf16_tflops, size) if family == "sotazen"
                                    else linedra_kernels(hbm_gbs, bf16_tflops, size) if family == "linedra"
+                                   else dozotar_kernels(hbm_gbs, bf16_tflops, size) if family == "dozotar"
                                    else dirurax_kernels(hbm_gbs, size))
         say(f"{size} kernels: {result['kernels'][size]}")
     clocks.stop()
@@ -1246,7 +1460,7 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=CONTEXT, help="with --only: context the decode ends at")
     ap.add_argument("--prompt-tokens", type=int, default=PREFILL_TOKENS,
                     help="with --only prefill: length of the prompt, computed in one step (up to 8192)")
-    ap.add_argument("--family", default="llama", choices=["llama", "dirurax", "pikalix", "sotazen", "linedra"],
+    ap.add_argument("--family", default="llama", choices=["llama", "dirurax", "pikalix", "sotazen", "linedra", "dozotar"],
                     help="dirurax, pikalix: that family's prefill and decode at a few sizes beside Llama models of equal size, "
                          "and its kernels alone (one JSON line of its own; the default workload is unchanged)")
     ap.add_argument("--size", default="", help="with --family dirurax or pikalix: sizes to run, with commas (default: all)")
@@ -1261,7 +1475,7 @@ def main() -> int:
         return 0
     args.warmup = max(args.warmup, 3)
     args.steps = max(args.steps, 2)
-    if args.family in ("dirurax", "pikalix", "sotazen", "linedra"):
+    if args.family in ("dirurax", "pikalix", "sotazen", "linedra", "dozotar"):
         return family_bench(args)
 
     import torch

@@ -81,10 +81,12 @@ struct Geometry {
     int window;            // 0: every earlier key
     int sink;              // the denominator holds exp(sink_values[h]) (null: exp(0)) besides the keys' terms
     int splits;            // ranges the key tiles of a CTA are cut into (grid z); > 1: results go through `part`
+    int page_shift;        // log2 of page_size where that is a power of two, else -1
     float scale, softcap;  // softcap 0: scores are not capped
     const float* slopes;   // slopes[h] * (query position - key position) is taken off head h's scores (null: no such bias)
     const float* bias;     // bias[h * bias_len + min(query position - key position, bias_len - 1)] is added to head h's scores (null: none)
     int bias_len;
+    int bias_span, bias_stride;    // bias in shared memory: distances it covers there, floats from one head to the next
     int block;             // > 0: a query sees only keys of its own block of that many positions (counted from 0)
 };
 
@@ -93,7 +95,7 @@ struct Geometry {
 template <bool VIK>
 __device__ __forceinline__ void load_tile(bf16* Ks, bf16* Vs, const bf16* __restrict__ cache, const int* __restrict__ bt,
                                           int k0, int k_lo, int k_hi, size_t page_elems, size_t k_base, size_t v_base,
-                                          int page_size) {
+                                          int page_size, int page_shift) {
     constexpr int PIECES = KCH + (VIK ? 0 : VCH);
     for (int c = threadIdx.x; c < KT * PIECES; c += THREADS) {
         const int kk = c / PIECES, ch = c - kk * PIECES;
@@ -101,7 +103,7 @@ __device__ __forceinline__ void load_tile(bf16* Ks, bf16* Vs, const bf16* __rest
         const bool ok = key >= k_lo && key < k_hi;
         const bf16* src = cache;
         if (ok) {
-            const int blk = key / page_size, off = key - blk * page_size;
+            const int blk = page_shift >= 0 ? key >> page_shift : key / page_size, off = key - blk * page_size;
             const bf16* page = cache + (size_t)bt[blk] * page_elems;
             src = ch < KCH ? page + k_base + (size_t)off * HD + ch * 8 : page + v_base + (size_t)off * VD + (ch - KCH) * 8;
         }
@@ -110,8 +112,10 @@ __device__ __forceinline__ void load_tile(bf16* Ks, bf16* Vs, const bf16* __rest
     }
 }
 
-// BIAS: the scores carry the learned distance bias (an instantiation of its own: it costs registers)
-template <typename TO, bool VIK, bool BIAS>
+// BIAS: the scores carry the learned distance bias (instantiations of their own: it costs registers).  1: every distance a
+// tile can meet lies in shared memory, a row a head, in units of log2, so that a score costs one load at a fixed offset and
+// the multiply-add that scales it; 2: the table is read where it lies, the distance clamped to its end.
+template <typename TO, bool VIK, int BIAS>
 __global__ void __launch_bounds__(THREADS, VD <= 128 ? (VIK ? 4 : 3) : 1)      // values to 128 wide: three or four CTAs an SM
 attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__ out, int out_stride,
                       const bf16* __restrict__ cache, const int* __restrict__ block_table, int table_stride,
@@ -167,9 +171,19 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
     const size_t v_base = (size_t)Hk * gm.page_size * HD + (size_t)kvh * gm.page_size * VD;
 
     if (t_begin < t_end)
-        load_tile<VIK>(KVs, KVs + KT * KROW, cache, bt, t_begin * KT, lo_tile, p_last + 1, page_elems, k_base, v_base, gm.page_size);
+        load_tile<VIK>(KVs, KVs + KT * KROW, cache, bt, t_begin * KT, lo_tile, p_last + 1, page_elems, k_base, v_base, gm.page_size, gm.page_shift);
     cp_async_commit();
     __syncthreads();                                          // Qs is written
+
+    const int p_warp_first = p_first + (warp * 16) / Gc;     // position of the warp's first row
+    float* Bs = reinterpret_cast<float*>(KVs + 2 * BUF);      // BIAS 1: [Gc][bias_stride]
+    if (BIAS == 1) {
+        const int need = min(gm.bias_span, p_last - lo_tile + 1);
+        for (int hh = 0; hh < nheads; ++hh)
+            for (int i = tid; i < need; i += THREADS)
+                Bs[hh * gm.bias_stride + i] = gm.bias[(size_t)head_of(hh) * gm.bias_len + min(i, gm.bias_len - 1)] * LOG2E;
+        // (read after the barrier that every tile has)
+    }
 
     // this thread's two rows: 16 * warp + lane / 4 and that + 8
     int p_row[2], lo_row[2];
@@ -181,9 +195,9 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
         const int r = warp * 16 + (lane >> 2) + 8 * i;
         const int jj = r / Gc, hh = r - jj * Gc;
         ok_row[i] = jj < ntok && hh < nheads;
-        if (gm.slopes && ok_row[i]) slope[i] = gm.slopes[head_of(hh)];
-        if (BIAS && ok_row[i]) bias_row[i] = head_of(hh) * gm.bias_len;
-        p_row[i] = p_first + jj;
+        if (gm.slopes && ok_row[i]) slope[i] = gm.slopes[head_of(hh)] * LOG2E;
+        if (BIAS && ok_row[i]) bias_row[i] = BIAS == 1 ? hh * gm.bias_stride : head_of(hh) * gm.bias_len;
+        p_row[i] = ok_row[i] ? p_first + jj : p_warp_first;
         lo_row[i] = gm.window > 0 ? max(0, p_row[i] - gm.window + 1) : 0;
         if (gm.block > 0) lo_row[i] = max(lo_row[i], p_row[i] / gm.block * gm.block);
         m[i] = -INFINITY;
@@ -194,6 +208,11 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
             if ((lane & 3) == 0) l[i] = 1.f;
         }
     }
+    // tiles between these two need no mask: the warp's first row sees their last key, its last row their first
+    const int p_warp_last = p_first + min(ntok - 1, (warp * 16 + 15) / Gc);
+    int lo_warp = gm.window > 0 ? max(0, p_warp_last - gm.window + 1) : 0;
+    if (gm.block > 0) lo_warp = max(lo_warp, p_warp_last / gm.block * gm.block);
+    const float scale2 = gm.scale * LOG2E;
     const bool warp_active = (warp * 16) / Gc < ntok;        // rows beyond the tile's tokens: nothing to do
 
     unsigned qf[QREG ? KS : 1][4];
@@ -213,7 +232,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
         constexpr int VSTRIDE = VIK ? KROW : VROW;
         if (t + 1 < t_end) {
             bf16* Kn = KVs + (buf ^ 1) * BUF;
-            load_tile<VIK>(Kn, Kn + KT * KROW, cache, bt, (t + 1) * KT, lo_tile, p_last + 1, page_elems, k_base, v_base, gm.page_size);
+            load_tile<VIK>(Kn, Kn + KT * KROW, cache, bt, (t + 1) * KT, lo_tile, p_last + 1, page_elems, k_base, v_base, gm.page_size, gm.page_shift);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -239,19 +258,42 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, TO* __restrict__
             // scale, cap, mask; everything from here on in units of log2
             const int key0 = t * KT + (lane & 3) * 2;
             float mx[2] = {-INFINITY, -INFINITY};
+            if (t * KT + KT - 1 <= p_warp_first && t * KT >= lo_warp && !(gm.softcap > 0.f) && !gm.slopes) {
 #pragma unroll
-            for (int n = 0; n < KT / 8; ++n) {
+                for (int i = 0; i < 2; ++i) {
+                    const int d0 = p_row[i] - key0;           // distance of the thread's first key
+                    const float* bp = BIAS == 1 ? Bs + bias_row[i] + d0 : nullptr;
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int key = key0 + n * 8 + (e & 1);
-                    const int i = e >> 1;
-                    float sc = s[n][e] * gm.scale;
-                    if (gm.softcap > 0.f) sc = gm.softcap * tanhf(sc / gm.softcap);
-                    sc -= slope[i] * (float)(p_row[i] - key);
-                    if (BIAS) sc += __ldg(gm.bias + bias_row[i] + max(0, min(p_row[i] - key, gm.bias_len - 1)));
-                    const bool seen = ok_row[i] && key <= p_row[i] && key >= lo_row[i];
-                    s[n][e] = seen ? sc * LOG2E : -INFINITY;
-                    mx[i] = fmaxf(mx[i], s[n][e]);
+                    for (int n = 0; n < KT / 8; ++n) {
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) {
+                            float sc = s[n][2 * i + e] * scale2;
+                            if (BIAS == 1) sc = fmaf(s[n][2 * i + e], scale2, bp[-(n * 8 + e)]);
+                            if (BIAS == 2)
+                                sc = fmaf(s[n][2 * i + e], scale2, __ldg(gm.bias + bias_row[i] + min(d0 - n * 8 - e, gm.bias_len - 1)) * LOG2E);
+                            s[n][2 * i + e] = sc;
+                            mx[i] = fmaxf(mx[i], sc);
+                        }
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int n = 0; n < KT / 8; ++n) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int key = key0 + n * 8 + (e & 1);
+                        const int i = e >> 1;
+                        const bool seen = ok_row[i] && key <= p_row[i] && key >= lo_row[i];
+                        float sc;
+                        if (gm.softcap > 0.f) sc = gm.softcap * tanhf(s[n][e] * gm.scale / gm.softcap) * LOG2E;
+                        else sc = s[n][e] * scale2;
+                        sc -= slope[i] * (float)(p_row[i] - key);
+                        if (BIAS == 1 && seen) sc = fmaf(s[n][e], scale2, Bs[bias_row[i] + p_row[i] - key]);
+                        if (BIAS == 2 && seen)
+                            sc = fmaf(s[n][e], scale2, __ldg(gm.bias + bias_row[i] + min(p_row[i] - key, gm.bias_len - 1)) * LOG2E);
+                        s[n][e] = seen ? sc : -INFINITY;
+                        mx[i] = fmaxf(mx[i], s[n][e]);
+                    }
                 }
             }
             float alpha[2], muse[2];
@@ -415,14 +457,17 @@ attention_rows_merge_kernel(const float* __restrict__ part, TO* __restrict__ out
     }
 }
 
-template <typename TO, bool VIK, bool BIAS>
+constexpr size_t BIAS_SMEM = 24 * 1024;        // most shared memory the bias takes
+template <typename TO, bool VIK, int BIAS>
 int launch(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
            int table_stride, const int* cu_q, const int* kv_len, const int* tile_entry, const int* tile_tok0,
            int n_tiles, const float* sink_values, float* part, const Geometry& gm, cudaStream_t s) {
     static bool configured = false;
-    const size_t smem = ((size_t)MT * KROW + 2 * ((size_t)KT * KROW + (VIK ? 0 : (size_t)KT * VROW))) * sizeof(bf16);
+    constexpr size_t base = ((size_t)MT * KROW + 2 * ((size_t)KT * KROW + (VIK ? 0 : (size_t)KT * VROW))) * sizeof(bf16);
+    const size_t smem = base + (BIAS == 1 ? (size_t)gm.Gc * gm.bias_stride * sizeof(float) : 0);
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                             (int)(base + (BIAS == 1 ? BIAS_SMEM : 0)));
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
@@ -459,8 +504,8 @@ RI_API int ri_attention_rows_ctas_per_sm(int value_in_key, int out_f32) {
     cudaError_t e = cudaErrorInvalidValue;
 #define RI_ROWS_OCC(TO, VIK) do { \
         const size_t smem = ((size_t)MT * KROW + 2 * ((size_t)KT * KROW + (VIK ? 0 : (size_t)KT * VROW))) * sizeof(bf16); \
-        e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attention_rows_kernel<TO, VIK, false>, THREADS, smem); \
+        e = cudaFuncSetAttribute(attention_rows_kernel<TO, VIK, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attention_rows_kernel<TO, VIK, 0>, THREADS, smem); \
     } while (0)
     if (value_in_key) {
         if constexpr (VD <= HD) { if (out_f32) RI_ROWS_OCC(float, true); else RI_ROWS_OCC(bf16, true); }
@@ -488,18 +533,28 @@ RI_API int ri_attention_rows(const void* q, int q_stride, void* out, int out_str
     const int gc = ri_attention_rows_heads_per_cta(Hq, Hkv, maps);
     if (gc <= 0 || (value_in_key && (maps != 1 || VD > HD)) || q_stride % 8) return (int)cudaErrorInvalidValue;
     const int G = Hq / (Hkv * maps);
-    Geometry gm{Hq, Hkv, maps, gc, (G + gc - 1) / gc, MT / gc, page_size, window, sink, splits, scale, softcap, slopes,
-                bias, bias_len, block};
+    Geometry gm{Hq, Hkv, maps, gc, (G + gc - 1) / gc, MT / gc, page_size, window, sink, splits, -1, scale, softcap, slopes,
+                bias, bias_len, 0, 0, block};
+    for (int sh = 0; sh < 20; ++sh)
+        if (page_size == 1 << sh) gm.page_shift = sh;
+    // distances a query can meet: the block's, the window's, or no bound
+    if (bias && (block > 0 || window > 0)) {
+        const int span = block > 0 && window > 0 ? (block < window ? block : window) : block > 0 ? block : window;
+        const int stride = (span + 31) / 32 * 32 + 8;         // heads 8 banks apart: the lanes of a warp read without conflict
+        if ((size_t)gc * stride * sizeof(float) <= BIAS_SMEM) { gm.bias_span = span; gm.bias_stride = stride; }
+    }
     cudaStream_t s = (cudaStream_t)stream;
     if (bias && value_in_key) return (int)cudaErrorNotSupported;
+    if (bias && (softcap > 0.f || slopes)) return (int)cudaErrorNotSupported;
 #define RI_ROWS_GO(TO, VIK, BIAS) launch<TO, VIK, BIAS>(q, q_stride, out, out_stride, cache, block_table, table_stride, cu_q, kv_len, \
                                             tile_entry, tile_tok0, n_tiles, sink_values, part, gm, s)
     if (value_in_key) {
-        if constexpr (VD <= HD) return out_f32 ? RI_ROWS_GO(float, true, false) : RI_ROWS_GO(bf16, true, false);
+        if constexpr (VD <= HD) return out_f32 ? RI_ROWS_GO(float, true, 0) : RI_ROWS_GO(bf16, true, 0);
         return (int)cudaErrorInvalidValue;
     }
-    if (bias) return out_f32 ? RI_ROWS_GO(float, false, true) : RI_ROWS_GO(bf16, false, true);
-    return out_f32 ? RI_ROWS_GO(float, false, false) : RI_ROWS_GO(bf16, false, false);
+    if (bias && gm.bias_span) return out_f32 ? RI_ROWS_GO(float, false, 1) : RI_ROWS_GO(bf16, false, 1);
+    if (bias) return out_f32 ? RI_ROWS_GO(float, false, 2) : RI_ROWS_GO(bf16, false, 2);
+    return out_f32 ? RI_ROWS_GO(float, false, 0) : RI_ROWS_GO(bf16, false, 0);
 #undef RI_ROWS_GO
 }
 

@@ -271,6 +271,88 @@ __global__ void short_conv_kernel(const TI* __restrict__ x, int x_stride, const 
     }
 }
 
+// The same for fp32 inputs of up to four taps whose channels come in fours (16-byte rows): a thread owns four channels of a
+// chunk of CONV4_CHUNK tokens, all its loads in flight at once.  Taps beyond the convolution's are zeros in front.
+constexpr int CONV4_TAPS = 4, CONV4_CHUNK = 8;
+
+template <typename TO>
+__global__ void __launch_bounds__(128)
+short_conv4_kernel(const float* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias,
+                   float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
+                   TO* __restrict__ out, int out_stride, int C, int taps, int residual, const float* __restrict__ in_bias,
+                   int silu, StepSizes ss) {
+    pdl_trigger();
+    pdl_wait();
+    const int e = blockIdx.y;
+    const int t0 = cu_q[e], q_len = cu_q[e + 1] - t0;
+    const int i0 = blockIdx.z * CONV4_CHUNK;
+    if (i0 >= q_len) return;
+    const int i1 = min(q_len, i0 + CONV4_CHUNK);
+    const int c4 = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c4 * 4 >= C) {
+        const int h = c4 - C / 4;                             // behind the channels: a thread a head of the step sizes
+        if (h >= ss.H) return;
+        const float a = expf(ss.a_log[h]), b = ss.bias[h];
+        for (int i = i0; i < i1; ++i) {
+            const float v = x[(size_t)(t0 + i) * x_stride + C + h] + b;
+            const float dt = v > 20.f ? v + log1pf(expf(-v)) : log1pf(expf(v));
+            ss.dt[(size_t)(t0 + i) * ss.H + h] = dt;
+            ss.decay[(size_t)(t0 + i) * ss.H + h] = expf(-a * dt);
+        }
+        return;
+    }
+    const int c = c4 * 4, back = taps - 1;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float* st = state + ((size_t)state_slots[e] * back) * C + c;
+    const float4 ib = in_bias ? load4<float>(in_bias + c) : zero;
+    auto add = [](float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); };
+    // in[k]: the input at chunk place k - (CONV4_TAPS - 1); the places before the entry's start come from the state
+    float4 in[CONV4_TAPS - 1 + CONV4_CHUNK];
+#pragma unroll
+    for (int k = 0; k < CONV4_TAPS - 1 + CONV4_CHUNK; ++k) {
+        const int i = i0 + k - (CONV4_TAPS - 1);
+        in[k] = zero;
+        if (i >= 0) {
+            if (i < i1) in[k] = add(load4<float>(x + (size_t)(t0 + i) * x_stride + c), ib);
+        } else if (back + i >= 0) {
+            in[k] = load4<float>(st + (size_t)(back + i) * C);
+        }
+    }
+    float4 wt[CONV4_TAPS];                                    // wt[j]: the tap CONV4_TAPS - 1 - j tokens back, a channel a component
+#pragma unroll
+    for (int j = 0; j < CONV4_TAPS; ++j) {
+        const int tap = j - (CONV4_TAPS - taps);
+        wt[j] = tap < 0 ? zero : make_float4(w[(size_t)c * taps + tap], w[(size_t)(c + 1) * taps + tap],
+                                             w[(size_t)(c + 2) * taps + tap], w[(size_t)(c + 3) * taps + tap]);
+    }
+    const float4 b = bias ? load4<float>(bias + c) : zero;
+    auto act = [&](float y) { return silu ? y / (1.0f + expf(-y)) : y; };
+#pragma unroll
+    for (int k = 0; k < CONV4_CHUNK; ++k) {
+        if (i0 + k >= i1) break;
+        const float4 cur = in[k + CONV4_TAPS - 1];
+        float4 y = residual ? add(b, cur) : b;
+#pragma unroll
+        for (int j = CONV4_TAPS - 1; j >= 0; --j) {           // from the current token back, as the general kernel adds
+            const float4 v = in[k + j];
+            y = make_float4(fmaf(wt[j].x, v.x, y.x), fmaf(wt[j].y, v.y, y.y), fmaf(wt[j].z, v.z, y.z), fmaf(wt[j].w, v.w, y.w));
+        }
+        store4<TO>(out + (size_t)(t0 + i0 + k) * out_stride + c, make_float4(act(y.x), act(y.y), act(y.z), act(y.w)));
+    }
+    if (i0 != 0 || back == 0) return;
+    // the entry's last inputs; the first chunk's thread is the only one that reads or writes the channel's state
+    float4 last[CONV4_TAPS - 1];
+#pragma unroll
+    for (int k = 0; k < CONV4_TAPS - 1; ++k) {
+        const int i = q_len - back + k;
+        last[k] = zero;
+        if (k < back) last[k] = i >= 0 ? add(load4<float>(x + (size_t)(t0 + i) * x_stride + c), ib) : load4<float>(st + (size_t)(back + i) * C);
+    }
+#pragma unroll
+    for (int k = 0; k < CONV4_TAPS - 1; ++k)
+        if (k < back) store4<float>(st + (size_t)k * C, last[k]);
+}
+
 // ------------------------------------------------------------------ gates of the real-gated linear recurrent unit
 // u [T][C] fp32 in `blocks` equal parts of bs channels; wa, wi [blocks][bs][bs] ([out][in]), ba, bi [C]:
 //   r = sigmoid(wa[b] u_b + ba),  i = sigmoid(wi[b] u_b + bi),  log a = -decay_scale * r * softplus(lam),
@@ -550,6 +632,19 @@ RI_API int ri_short_conv(const void* x, int x_dtype, int x_stride, const float* 
         return (int)cudaErrorInvalidValue;
     const StepSizes sizes{dt_bias, a_log, dt, decay, dt_heads};
     cudaStream_t s = (cudaStream_t)stream;
+    auto at16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const int osize = out_dtype == RI_BF16 ? 2 : 4;
+    if (x_dtype == RI_F32 && taps <= CONV4_TAPS && C % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 && at16(x) && at16(state) &&
+        ((uintptr_t)out % (4 * osize)) == 0 && (!bias || at16(bias)) && (!in_bias || at16(in_bias))) {
+        const dim3 g4((C / 4 + dt_heads + 127) / 128, n_entries, (max_q_len + CONV4_CHUNK - 1) / CONV4_CHUNK);
+        if (out_dtype == RI_BF16)
+            RI_CHECKED(ri_launch(short_conv4_kernel<bf16>, g4, dim3(128), 0, s, (const float*)x, x_stride, w, bias, state, cu_q, state_slots,
+                                 (bf16*)out, out_stride, C, taps, residual, in_bias, silu, sizes));
+        else
+            RI_CHECKED(ri_launch(short_conv4_kernel<float>, g4, dim3(128), 0, s, (const float*)x, x_stride, w, bias, state, cu_q, state_slots,
+                                 (float*)out, out_stride, C, taps, residual, in_bias, silu, sizes));
+        return ri_launch_status();
+    }
     const dim3 grid((C + dt_heads + 127) / 128, n_entries, (max_q_len + CONV_CHUNK - 1) / CONV_CHUNK);
 #define RI_SC(TI, TO) RI_CHECKED(ri_launch(short_conv_kernel<TI, TO>, grid, dim3(128), 0, s, (const TI*)x, x_stride, w, bias, \
         state, cu_q, state_slots, (TO*)out, out_stride, C, taps, residual, in_bias, silu, sizes))

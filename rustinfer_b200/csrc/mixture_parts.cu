@@ -29,10 +29,11 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
     }
 }
 
-constexpr int ROUTE_WARPS = 4, ROUTE_CHUNK = 8;
+// TT tokens a CTA (a row of the router's matrix is read once for them), each warp a few experts at a time.
+constexpr int ROUTE_CHUNK = 8;
 
-template <typename TX>
-__global__ void __launch_bounds__(32 * ROUTE_WARPS)
+template <typename TX, int TT>
+__global__ void __launch_bounds__(512)
 moe_route_kernel(const float* __restrict__ z, const TX* __restrict__ x, const float* __restrict__ router,
                  int d, const float* __restrict__ correction, int T, int E,
                  int top, int n_groups, int keep, int renorm, int* __restrict__ ids,
@@ -42,36 +43,52 @@ moe_route_kernel(const float* __restrict__ z, const TX* __restrict__ x, const fl
     pdl_wait();
     extern __shared__ float sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x;
+    const int warps = blockDim.x >> 5, t0 = blockIdx.x * TT;
     // gate (with x): the router's matrix has one row more, whose product's sigmoid goes to gate[t]
     const int rows = E + (gate && x ? 1 : 0);
-    float* s = sm;                                         // [rows] scores
-    float* c = s + rows;                                   // [E] choice scores
-    float* gs = c + E;                                     // [n_groups] group scores
+    const int per_token = rows + E + n_groups;
     if (x) {
-        // the logits: the warps share the experts, eight at a time; a lane takes every 32nd term of all eight
-        // sums (x is read once for them), then the lanes' parts meet in a butterfly
-        const TX* xr = x + (size_t)t * d;
-        for (int e0 = warp * ROUTE_CHUNK; e0 < rows; e0 += ROUTE_WARPS * ROUTE_CHUNK) {
-            float acc[ROUTE_CHUNK];
+        // the logits: the warps share the experts, a few (at most eight) at a time; a lane takes every 32nd term of
+        // their sums for every token (x and the matrix are read once for all), then the lanes' parts meet in a butterfly
+        const int ch = min(ROUTE_CHUNK, (rows + warps - 1) / warps);
+        for (int e0 = warp * ch; e0 < rows; e0 += warps * ch) {
+            const int ne = min(ch, rows - e0);
+            float acc[ROUTE_CHUNK][TT];
 #pragma unroll
-            for (int j = 0; j < ROUTE_CHUNK; ++j) acc[j] = 0.f;
+            for (int j = 0; j < ROUTE_CHUNK; ++j)
+#pragma unroll
+                for (int k = 0; k < TT; ++k) acc[j][k] = 0.f;
 #pragma unroll 4
             for (int i = lane; i < d; i += 32) {
-                const float xv = to_f32<TX>(xr[i]);
+                float xv[TT];
+#pragma unroll
+                for (int k = 0; k < TT; ++k) xv[k] = to_f32<TX>(x[(size_t)min(t0 + k, T - 1) * d + i]);
 #pragma unroll
                 for (int j = 0; j < ROUTE_CHUNK; ++j)
-                    if (e0 + j < rows) acc[j] = fmaf(xv, router[(size_t)(e0 + j) * d + i], acc[j]);
+                    if (j < ne) {
+                        const float w = router[(size_t)(e0 + j) * d + i];
+#pragma unroll
+                        for (int k = 0; k < TT; ++k) acc[j][k] = fmaf(xv[k], w, acc[j][k]);
+                    }
             }
 #pragma unroll
-            for (int j = 0; j < ROUTE_CHUNK; ++j) {
-                const float dot = warp_sum(acc[j]);
-                if (lane == 0 && e0 + j < rows) s[e0 + j] = dot;
-            }
+            for (int j = 0; j < ROUTE_CHUNK; ++j)
+                if (j < ne) {
+#pragma unroll
+                    for (int k = 0; k < TT; ++k) {
+                        const float dot = warp_sum(acc[j][k]);
+                        if (lane == 0) sm[k * per_token + e0 + j] = dot;
+                    }
+                }
         }
         __syncthreads();
     }
-    if (warp != 0) return;                                 // the choice is one warp's work
+    // the choice is one warp's work a token
+    const int t = t0 + warp;
+    if (warp >= TT || t >= T) return;
+    float* s = sm + warp * per_token;                      // [rows] scores
+    float* c = s + rows;                                   // [E] choice scores
+    float* gs = c + E;                                     // [n_groups] group scores
     if (gate && x && lane == 0) gate[t] = 1.0f / (1.0f + expf(-s[E]));
     float zmx = -INFINITY, zsum = 0.f;                     // of the softmax over all experts
     if (score == 2) {
@@ -497,19 +514,21 @@ RI_API int ri_moe_route(const float* z, const void* x, int x_dtype, const float*
     if (score < 0 || score > 2 || (gate && !x)) return (int)cudaErrorInvalidValue;
     if (E <= 0 || top <= 0 || top > E || top > 32 || (n_groups > 0 && (E % n_groups || keep <= 0 || keep > n_groups)))
         return (int)cudaErrorInvalidValue;
-    const int warps = ROUTE_WARPS;
-    const size_t smem = (size_t)(2 * E + 1 + (n_groups > 0 ? n_groups : 0)) * sizeof(float);
+    // few tokens: a CTA each with many warps on the router's rows; many: four tokens a CTA
+    const int rows = E + (gate ? 1 : 0);
+    const bool tiled = x && T > 4 * ri_device_sms();
+    const int tt = tiled ? 4 : 1;
+    const int warps = tiled ? 8 : x ? (rows < 16 ? rows : 16) : 1;
+    const size_t smem = (size_t)tt * (rows + E + (n_groups > 0 ? n_groups : 0)) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     if ((z == nullptr) == (x == nullptr) || (x && !router)) return (int)cudaErrorInvalidValue;
-    const dim3 grid(T);
-    if (x && x_dtype == RI_BF16)
-        RI_CHECKED(ri_launch(moe_route_kernel<bf16>, grid, dim3(32 * warps), smem, (cudaStream_t)stream, z, (const bf16*)x, router, d,
-                             correction, T, E, top, n_groups > 0 ? n_groups : 0, keep, renorm, ids, weights, counts, score,
-                             group_max, renorm_eps, gate));
-    else
-        RI_CHECKED(ri_launch(moe_route_kernel<float>, grid, dim3(32 * warps), smem, (cudaStream_t)stream, z, (const float*)x, router, d,
-                             correction, T, E, top, n_groups > 0 ? n_groups : 0, keep, renorm, ids, weights, counts, score,
-                             group_max, renorm_eps, gate));
+    const dim3 grid((T + tt - 1) / tt);
+#define RI_MR(TX, TT) RI_CHECKED(ri_launch(moe_route_kernel<TX, TT>, grid, dim3(32 * warps), smem, (cudaStream_t)stream, z, (const TX*)x, router, d, \
+                                           correction, T, E, top, n_groups > 0 ? n_groups : 0, keep, renorm, ids, weights, counts, score, \
+                                           group_max, renorm_eps, gate))
+    if (x && x_dtype == RI_BF16) { if (tiled) RI_MR(bf16, 4); else RI_MR(bf16, 1); }
+    else { if (tiled) RI_MR(float, 4); else RI_MR(float, 1); }
+#undef RI_MR
     return ri_launch_status();
 }
 

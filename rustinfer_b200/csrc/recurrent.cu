@@ -141,18 +141,20 @@ __device__ __forceinline__ float4 ld4(const bf16* p) {
 __device__ __forceinline__ float4 scaled(float4 v, float s) { return make_float4(v.x * s, v.y * s, v.z * s, v.w * s); }
 
 // the lane's rows of its C columns: column j of the tile at sp + j * DKP
-__device__ __forceinline__ void load_state(float (&S)[C][NR], const float* sp, const bool (&ok)[C]) {
+template <int N>
+__device__ __forceinline__ void load_state(float (&S)[N][NR], const float* sp, const bool (&ok)[N]) {
 #pragma unroll
-    for (int j = 0; j < C; ++j)
+    for (int j = 0; j < N; ++j)
 #pragma unroll
         for (int m = 0; m < NR / 4; ++m) {
             const float4 x = ok[j] ? reinterpret_cast<const float4*>(sp + (size_t)j * DKP)[m] : make_float4(0.f, 0.f, 0.f, 0.f);
             S[j][4 * m] = x.x; S[j][4 * m + 1] = x.y; S[j][4 * m + 2] = x.z; S[j][4 * m + 3] = x.w;
         }
 }
-__device__ __forceinline__ void store_state(const float (&S)[C][NR], float* sp, const bool (&ok)[C]) {
+template <int N>
+__device__ __forceinline__ void store_state(const float (&S)[N][NR], float* sp, const bool (&ok)[N]) {
 #pragma unroll
-    for (int j = 0; j < C; ++j)
+    for (int j = 0; j < N; ++j)
         if (ok[j]) {
 #pragma unroll
             for (int m = 0; m < NR / 4; ++m)
@@ -578,11 +580,18 @@ delta_scan_kernel(const TA* __restrict__ r, int r_stride, const TA* __restrict__
 // As the gated walk, but a token's decay is one number a head, a_t, its values may be multiplied by another, g_t, and
 // heads share keys and queries in groups of `share` (head h reads key head h / share):
 //   S <- a S + k (g v);   o += S q
+// CC: columns a lane holds; fewer columns make more CTAs, for walks whose CTAs would not fill the SMs (a column's sums
+// are the same whatever CC is).
+template <int CC> struct HeadShape {
+    static constexpr int COLS = WORKERS / R * CC;            // value channels per CTA
+    static constexpr int PERV = (TC * COLS + WORKERS - 1) / WORKERS;
+    static constexpr int HALF = 2 * TC * ROWLEN + TC * COLS + 2 * TC;      // q, k, v, decays, gains
+};
+template <int CC>
 struct HeadHalf {
     float *q, *k, *v, *a;
-    __device__ HeadHalf(float* base) : q(base), k(base + TC * ROWLEN), v(base + 2 * TC * ROWLEN), a(v + TC * COLS) {}
+    __device__ HeadHalf(float* base) : q(base), k(base + TC * ROWLEN), v(base + 2 * TC * ROWLEN), a(v + TC * HeadShape<CC>::COLS) {}
 };
-constexpr int HEAD_HALF = 2 * TC * ROWLEN + TC * COLS + TC;
 
 __device__ __forceinline__ void head_rows(float* S, float a, const float4& k, const float4& q, float vj, float& o0, float& o1) {
     S[0] = fmaf(a, S[0], k.x * vj);
@@ -595,24 +604,82 @@ __device__ __forceinline__ void head_rows(float* S, float a, const float4& k, co
     o1 = fmaf(S[3], q.w, o1);
 }
 
-__device__ __forceinline__ void head_token(float (&S)[C][NR], const HeadHalf& b, int tok, int rg, int cg, float (&part)[C]) {
-    const float4* k4 = reinterpret_cast<const float4*>(b.k + tok * ROWLEN + rg * NRP);
-    const float4* q4 = reinterpret_cast<const float4*>(b.q + tok * ROWLEN + rg * NRP);
-    const float a = b.a[tok];
-    float vj[C], o0[C], o1[C];
+// Rows are kept in pairs: the packed multiply-add of two floats does both halves with the rounding of the scalar one, so
+// a walk's state has the bits the single-token kernel gives it with head_rows.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+    f32x2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 d) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(d));
+    return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+template <int N>
+__device__ __forceinline__ void load_pairs(f32x2 (&S)[N][NR / 2], const float* sp, const bool (&ok)[N]) {
 #pragma unroll
-    for (int j = 0; j < C; ++j) {
-        vj[j] = b.v[tok * COLS + cg * C + j];
-        o0[j] = o1[j] = 0.f;
+    for (int j = 0; j < N; ++j)
+#pragma unroll
+        for (int m = 0; m < NR / 4; ++m) {
+            const float4 x = ok[j] ? reinterpret_cast<const float4*>(sp + (size_t)j * DKP)[m] : make_float4(0.f, 0.f, 0.f, 0.f);
+            S[j][2 * m] = pack2(x.x, x.y);
+            S[j][2 * m + 1] = pack2(x.z, x.w);
+        }
+}
+template <int N>
+__device__ __forceinline__ void store_pairs(const f32x2 (&S)[N][NR / 2], float* sp, const bool (&ok)[N]) {
+#pragma unroll
+    for (int j = 0; j < N; ++j)
+        if (ok[j]) {
+#pragma unroll
+            for (int m = 0; m < NR / 4; ++m) {
+                const float2 lo = unpack2(S[j][2 * m]), hi = unpack2(S[j][2 * m + 1]);
+                reinterpret_cast<float4*>(sp + (size_t)j * DKP)[m] = make_float4(lo.x, lo.y, hi.x, hi.y);
+            }
+        }
+}
+
+template <int CC>
+__device__ __forceinline__ void head_token(f32x2 (&S)[CC][NR / 2], const HeadHalf<CC>& b, int tok, int rg, int cg, float (&part)[CC]) {
+    const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(b.k + tok * ROWLEN + rg * NRP);
+    const ulonglong2* q2 = reinterpret_cast<const ulonglong2*>(b.q + tok * ROWLEN + rg * NRP);
+    const float a = b.a[tok], g = b.a[TC + tok];
+    const f32x2 aa = pack2(a, a);
+    f32x2 vv[CC], o[CC];
+#pragma unroll
+    for (int j = 0; j < CC; ++j) {
+        const float v = g * b.v[tok * HeadShape<CC>::COLS + cg * CC + j];
+        vv[j] = pack2(v, v);
+        o[j] = 0ull;
     }
 #pragma unroll
     for (int m = 0; m < NR / 4; ++m) {
-        const float4 kk = k4[m], qq = q4[m];
+        const ulonglong2 kk = k2[m], qq = q2[m];
 #pragma unroll
-        for (int j = 0; j < C; ++j) head_rows(&S[j][4 * m], a, kk, qq, vj[j], o0[j], o1[j]);
+        for (int j = 0; j < CC; ++j) {
+            S[j][2 * m] = fma2(aa, S[j][2 * m], mul2(kk.x, vv[j]));
+            S[j][2 * m + 1] = fma2(aa, S[j][2 * m + 1], mul2(kk.y, vv[j]));
+            o[j] = fma2(S[j][2 * m], qq.x, o[j]);
+            o[j] = fma2(S[j][2 * m + 1], qq.y, o[j]);
+        }
     }
 #pragma unroll
-    for (int j = 0; j < C; ++j) part[j] = o0[j] + o1[j];
+    for (int j = 0; j < CC; ++j) {
+        const float2 p = unpack2(o[j]);
+        part[j] = p.x + p.y;
+    }
 }
 
 // q, k: [T, >= H/share*DK] with row strides; v: [T, >= H*dv]; decay: fp32, decay[t * a_stride + h] (a_stride 0: the same for
@@ -626,6 +693,7 @@ head_scan_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ 
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float smem[];
+    constexpr int CC = C, COLS = HeadShape<CC>::COLS, PERV = HeadShape<CC>::PERV, HALF = HeadShape<CC>::HALF;
     const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS;
     const int kh = h / share;
     const int tid = threadIdx.x;
@@ -635,23 +703,22 @@ head_scan_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ 
     const int t_begin = cu_q[b], t_end = cu_q[b + 1];
     const int rounds = (t_end - t_begin + TC - 1) / TC;
     if (DKP != DK) {                                         // rows beyond DK stay zero
-        for (int e = tid; e < 2 * HEAD_HALF; e += THREADS) smem[e] = 0.f;
+        for (int e = tid; e < 2 * HALF; e += THREADS) smem[e] = 0.f;
         __syncthreads();
     }
 
     auto stage = [&](int round) {
-        const HeadHalf hb(smem + (round & 1) * HEAD_HALF);
+        const HeadHalf<CC> hb(smem + (round & 1) * HALF);
         const int t0 = t_begin + round * TC, nt = min(TC, t_end - t0);
         float vv[PERV];
-        load_values(vv, v, v_stride, t0, nt, h, dv, c0, lt);
-        if (gain) {
 #pragma unroll
-            for (int j = 0; j < PERV; ++j) {
-                const int tok = min(lt + j * WORKERS, nt * COLS - 1) / COLS;
-                vv[j] *= gain[(size_t)(t0 + tok) * g_stride + h];
-            }
+        for (int j = 0; j < PERV; ++j) {
+            const int e = min(lt + j * WORKERS, nt * COLS - 1);
+            const int tok = e / COLS, c = min(e - tok * COLS, dv - 1 - c0);
+            vv[j] = ld(v, (size_t)(t0 + tok) * v_stride + (size_t)h * dv + c0 + c);
         }
         const float av = decay[(size_t)(t0 + min(lt, nt - 1)) * a_stride + h];
+        const float gv = gain ? gain[(size_t)(t0 + min(lt, nt - 1)) * g_stride + h] : 1.f;
         if (vec) {                                           // loads unconditional, as in the gated kernel
             float4 qv[PER4], kv[PER4];
 #pragma unroll
@@ -693,47 +760,54 @@ head_scan_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ 
                 }
             }
         }
-        store_values(hb.v, vv, nt, dv, c0, lt);
-        if (lt < nt) hb.a[lt] = av;
+#pragma unroll
+        for (int j = 0; j < PERV; ++j) {
+            const int e = lt + j * WORKERS;
+            if (e < nt * COLS) {
+                const int tok = e / COLS, c = e - tok * COLS;
+                hb.v[tok * COLS + c] = c0 + c < dv ? vv[j] : 0.f;
+            }
+        }
+        if (lt < nt) { hb.a[lt] = av; hb.a[TC + lt] = gv; }
     };
 
-    bool ok[C];
+    bool ok[CC];
 #pragma unroll
-    for (int j = 0; j < C; ++j) ok[j] = !loader && c0 + cg * C + j < dv;
+    for (int j = 0; j < CC; ++j) ok[j] = !loader && c0 + cg * CC + j < dv;
     float* sp = nullptr;
-    float S[C][NR];
+    f32x2 S[CC][NR / 2];
     if (loader) {
         if (rounds > 0) stage(0);
     } else {
-        sp = state + ((((size_t)state_slots[b] * H + h) * dv + c0 + cg * C) * DKP + rg * NR);
-        load_state(S, sp, ok);
+        sp = state + ((((size_t)state_slots[b] * H + h) * dv + c0 + cg * CC) * DKP + rg * NR);
+        load_pairs(S, sp, ok);
     }
     __syncthreads();
     for (int round = 0; round < rounds; ++round) {
         if (loader) {
             if (round + 1 < rounds) stage(round + 1);
         } else {
-            const HeadHalf hb(smem + (round & 1) * HEAD_HALF);
+            const HeadHalf<CC> hb(smem + (round & 1) * HALF);
             const int t0 = t_begin + round * TC, nt = min(TC, t_end - t0);
-            float* op = out + ((size_t)t0 * H + h) * dv + c0 + cg * C;
+            float* op = out + ((size_t)t0 * H + h) * dv + c0 + cg * CC;
             if (nt == TC) {
 #pragma unroll
                 for (int tb = 0; tb < TC; tb += TB) {        // the outputs' sums in batches, as in the gated kernel
-                    GroupSums<TB * C> sums;                  // value i * C + j: token tb + i, column j
+                    GroupSums<TB * CC> sums;                  // value i * CC + j: token tb + i, column j
 #pragma unroll
                     for (int i = 0; i < TB; ++i) {
-                        float part[C];
+                        float part[CC];
                         head_token(S, hb, tb + i, rg, cg, part);
 #pragma unroll
-                        for (int j = 0; j < C; ++j) sums.x[i * C + j] = part[j];
+                        for (int j = 0; j < CC; ++j) sums.x[i * CC + j] = part[j];
                     }
                     sums.run(rg);
                     if (sums.owner) {
 #pragma unroll
-                        for (int n = 0; n < TB * C; ++n) {
+                        for (int n = 0; n < TB * CC; ++n) {
                             if (n < sums.count) {
-                                const int idx = sums.first + n, i = idx / C, j = idx - i * C;
-                                if (c0 + cg * C + j < dv) op[(size_t)(tb + i) * H * dv + j] = sums.x[n];
+                                const int idx = sums.first + n, i = idx / CC, j = idx - i * CC;
+                                if (c0 + cg * CC + j < dv) op[(size_t)(tb + i) * H * dv + j] = sums.x[n];
                             }
                         }
                     }
@@ -741,10 +815,10 @@ head_scan_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ 
             } else {
 #pragma unroll 1
                 for (int tok = 0; tok < nt; ++tok) {
-                    float part[C];
+                    float part[CC];
                     head_token(S, hb, tok, rg, cg, part);
 #pragma unroll
-                    for (int j = 0; j < C; ++j) {
+                    for (int j = 0; j < CC; ++j) {
                         const float o = group_sum(part[j]);
                         if (rg == 0 && ok[j]) op[(size_t)tok * H * dv + j] = o;
                     }
@@ -753,7 +827,133 @@ head_scan_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ 
         }
         __syncthreads();
     }
-    if (!loader) store_state(S, sp, ok);
+    if (!loader) store_pairs(S, sp, ok);
+}
+
+// The same walk for fp32 inputs whose rows are whole 16-byte pieces: the vectors travel by cp.async into a ring of
+// HEAD_STAGES rounds, so that a trip to memory is as long as HEAD_STAGES - 1 rounds may take (with one round ahead the
+// walk waits for memory: 2 us a round of 16 tokens whatever the CTAs had to compute).  q_scale is applied to the sums.
+constexpr int HEAD_STAGES = 4;
+__device__ __forceinline__ void cp_async16(float* smem, const float* gmem, bool valid) {
+    const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+    const int n = valid ? 16 : 0;                            // 0 bytes read: zeros
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(s), "l"(gmem), "r"(n));
+}
+__device__ __forceinline__ void cp_async4(float* smem, const float* gmem) {
+    const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(s), "l"(gmem));
+}
+
+template <int CC>
+__global__ void __launch_bounds__(THREADS, DK <= 128 ? 2 : 1)
+head_scan_async_kernel(const float* __restrict__ q, int q_stride, const float* __restrict__ k, int k_stride,
+                       const float* __restrict__ v, int v_stride, const float* __restrict__ decay, int a_stride,
+                       const float* __restrict__ gain, int g_stride, float q_scale, float* __restrict__ out,
+                       float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
+                       int H, int dv, int share) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float smem[];
+    constexpr int COLS = HeadShape<CC>::COLS, HALF = HeadShape<CC>::HALF;
+    const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS;
+    const int kh = h / share;
+    const int tid = threadIdx.x;
+    const bool loader = tid >= WORKERS;
+    const int lt = tid - WORKERS;
+    const int cg = tid / R, rg = tid % R;
+    const int t_begin = cu_q[b], t_end = cu_q[b + 1];
+    const int rounds = (t_end - t_begin + TC - 1) / TC;
+    if (DKP != DK || !gain) {                                // rows beyond DK stay zero; without gains they stay one
+        for (int e = tid; e < HEAD_STAGES * HALF; e += THREADS) smem[e] = e % HALF >= HALF - TC ? 1.f : 0.f;
+        __syncthreads();
+    }
+    auto stage = [&](int round) {
+        const HeadHalf<CC> hb(smem + (round % HEAD_STAGES) * HALF);
+        const int t0 = t_begin + round * TC, nt = min(TC, t_end - t0);
+        constexpr int P = DK / 4 > 0 ? DK / 4 : 1;
+        for (int e = lt; e < nt * P; e += WORKERS) {
+            const int tok = e / P, i = (e - tok * P) * 4;
+            const size_t t = (size_t)(t0 + tok), c = (size_t)kh * DK + i;
+            const int at = tok * ROWLEN + row_at(i);
+            cp_async16(hb.q + at, q + t * q_stride + c, true);
+            cp_async16(hb.k + at, k + t * k_stride + c, true);
+        }
+        for (int e = lt; e < nt * (COLS / 4); e += WORKERS) {
+            const int tok = e / (COLS / 4), c = (e - tok * (COLS / 4)) * 4;
+            const bool in = c0 + c < dv;
+            cp_async16(hb.v + tok * COLS + c, in ? v + (size_t)(t0 + tok) * v_stride + (size_t)h * dv + c0 + c : v, in);
+        }
+        if (lt < nt) {
+            cp_async4(hb.a + lt, decay + (size_t)(t0 + lt) * a_stride + h);
+            if (gain) cp_async4(hb.a + TC + lt, gain + (size_t)(t0 + lt) * g_stride + h);
+        }
+    };
+    auto commit = [] { asm volatile("cp.async.commit_group;\n" ::); };
+    auto wait = [] { asm volatile("cp.async.wait_group %0;\n" ::"n"(HEAD_STAGES - 2)); };
+
+    bool ok[CC];
+#pragma unroll
+    for (int j = 0; j < CC; ++j) ok[j] = !loader && c0 + cg * CC + j < dv;
+    float* sp = nullptr;
+    f32x2 S[CC][NR / 2];
+    if (loader) {
+        for (int r = 0; r < HEAD_STAGES - 1; ++r) {
+            if (r < rounds) stage(r);
+            commit();
+        }
+        wait();
+    } else {
+        sp = state + ((((size_t)state_slots[b] * H + h) * dv + c0 + cg * CC) * DKP + rg * NR);
+        load_pairs(S, sp, ok);
+    }
+    __syncthreads();
+    for (int round = 0; round < rounds; ++round) {
+        if (loader) {
+            if (round + HEAD_STAGES - 1 < rounds) stage(round + HEAD_STAGES - 1);
+            commit();
+            wait();                                          // the next round has landed
+        } else {
+            const HeadHalf<CC> hb(smem + (round % HEAD_STAGES) * HALF);
+            const int t0 = t_begin + round * TC, nt = min(TC, t_end - t0);
+            float* op = out + ((size_t)t0 * H + h) * dv + c0 + cg * CC;
+            if (nt == TC) {
+#pragma unroll
+                for (int tb = 0; tb < TC; tb += TB) {
+                    GroupSums<TB * CC> sums;                 // value i * CC + j: token tb + i, column j
+#pragma unroll
+                    for (int i = 0; i < TB; ++i) {
+                        float part[CC];
+                        head_token(S, hb, tb + i, rg, cg, part);
+#pragma unroll
+                        for (int j = 0; j < CC; ++j) sums.x[i * CC + j] = part[j];
+                    }
+                    sums.run(rg);
+                    if (sums.owner) {
+#pragma unroll
+                        for (int n = 0; n < TB * CC; ++n) {
+                            if (n < sums.count) {
+                                const int idx = sums.first + n, i = idx / CC, j = idx - i * CC;
+                                if (c0 + cg * CC + j < dv) op[(size_t)(tb + i) * H * dv + j] = sums.x[n] * q_scale;
+                            }
+                        }
+                    }
+                }
+            } else {
+#pragma unroll 1
+                for (int tok = 0; tok < nt; ++tok) {
+                    float part[CC];
+                    head_token(S, hb, tok, rg, cg, part);
+#pragma unroll
+                    for (int j = 0; j < CC; ++j) {
+                        const float o = group_sum(part[j]);
+                        if (rg == 0 && ok[j]) op[(size_t)tok * H * dv + j] = o * q_scale;
+                    }
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (!loader) store_pairs(S, sp, ok);
 }
 
 // ------------------------------------------------------------- entries of a single token
@@ -1003,8 +1203,10 @@ RI_API int ri_head_scan(const void* q, int q_stride, const void* k, int k_stride
         return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid((dv + COLS - 1) / COLS, H, entries);
-    const size_t smem = 2 * (size_t)HEAD_HALF * sizeof(float);
     const int esize = act_dtype == RI_BF16 ? 2 : 4;
+    // columns a lane of the asynchronous walk: half as many where that does not yet fill the SMs once
+    const long long ctas = (long long)grid.x * grid.y * grid.z;
+    const bool narrow = 2 * ctas <= ri_device_sms();
     const int vec = DK % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && aligned4(q, esize) && aligned4(k, esize);
     const StepRotation ro{positions, cos_t, sin_t, rot, interleaved};
 #define RI_HS(TA) do { \
@@ -1014,13 +1216,27 @@ RI_API int ri_head_scan(const void* q, int q_stride, const void* k, int k_stride
         break; \
     } \
     static bool allowed = false; \
+    const size_t smem = 2 * (size_t)HeadShape<C>::HALF * sizeof(float); \
     if (!allowed) { RI_CHECKED(allow_shared(head_scan_kernel<TA>, smem)); allowed = true; } \
     RI_CHECKED(ri_launch(head_scan_kernel<TA>, grid, dim3(THREADS), smem, s, (const TA*)q, q_stride, (const TA*)k, k_stride, \
         (const TA*)v, v_stride, decay, a_stride, gain, g_stride, q_scale, out, state, cu_q, state_slots, H, dv, share, vec)); \
     } while (0)
+#define RI_HSA(CC) do { \
+    static bool allowed = false; \
+    const size_t smem = HEAD_STAGES * (size_t)HeadShape<CC>::HALF * sizeof(float); \
+    if (!allowed) { RI_CHECKED(allow_shared(head_scan_async_kernel<CC>, smem)); allowed = true; } \
+    const dim3 g((dv + HeadShape<CC>::COLS - 1) / HeadShape<CC>::COLS, H, entries); \
+    RI_CHECKED(ri_launch(head_scan_async_kernel<CC>, g, dim3(THREADS), smem, s, (const float*)q, q_stride, (const float*)k, k_stride, \
+        (const float*)v, v_stride, decay, a_stride, gain, g_stride, q_scale, out, state, cu_q, state_slots, H, dv, share)); \
+    return ri_launch_status(); } while (0)
+    if (!single && act_dtype == RI_F32 && vec && dv % 4 == 0 && v_stride % 4 == 0 && aligned4(v, 4)) {
+        if (narrow) RI_HSA(C / 2);
+        RI_HSA(C);
+    }
     if (act_dtype == RI_BF16) RI_HS(bf16);
     else RI_HS(float);
 #undef RI_HS
+#undef RI_HSA
     return ri_launch_status();
 }
 

@@ -179,13 +179,17 @@ __device__ __forceinline__ float conv_channel(const QkvConv& cv, int t, int c, i
     const int back = cv.taps - 1;
     const float* wc = cv.w + (size_t)c * cv.taps;
     float* st = cv.state + (size_t)cv.slots[t] * back * channels + c;
-    float y = wc[back] * x, prev = x;
-    for (int k = back - 1; k >= 0; --k) {
-        const float old = st[(size_t)k * channels];
-        y = fmaf(wc[k], old, y);
-        st[(size_t)k * channels] = prev;
-        prev = old;
-    }
+    constexpr int MAX_BACK = 7;
+    float old[MAX_BACK];                          // every load is issued before the first store
+#pragma unroll
+    for (int k = 0; k < MAX_BACK; ++k) old[k] = k < back ? st[(size_t)k * channels] : 0.f;
+    float y = wc[back] * x;
+#pragma unroll
+    for (int k = MAX_BACK - 1; k >= 0; --k)
+        if (k < back) y = fmaf(wc[k], old[k], y);
+#pragma unroll
+    for (int k = 0; k < MAX_BACK; ++k)
+        if (k < back) st[(size_t)k * channels] = k + 1 < back ? old[k + 1 < MAX_BACK ? k + 1 : k] : x;
     return y;
 }
 
@@ -334,7 +338,7 @@ RI_API int ri_qkv_prepare(const void* qkv, int in_dtype, int row_stride, const f
                           int has_kv, int page_size, int value_heads, const float* conv_w, float* conv_state,
                           const int* conv_slots, int conv_taps, void* stream) {
     if (tokens <= 0) return 0;
-    if (conv_w && (!conv_slots || conv_taps < 1 || (conv_taps > 1 && !conv_state))) return (int)cudaErrorInvalidValue;
+    if (conv_w && (!conv_slots || conv_taps < 1 || conv_taps > 8 || (conv_taps > 1 && !conv_state))) return (int)cudaErrorInvalidValue;
     const QkvConv cv{conv_w, conv_state, conv_slots, conv_taps};
     // with the convolution a step has few tokens and a thread waits for its channel's state: more threads a token
     const int threads = conv_w ? 1024 : 256;
