@@ -1057,10 +1057,31 @@ struct StepRotation {
     const float *cos_t, *sin_t;
     int rot, interleaved;
 };
+// vec: rows come in aligned fours, and so do the halves of a rotation.
 template <typename TA>
-__device__ __forceinline__ void rotated_rows_of(float4 (&x)[NR / 4], const TA* p, int rg, float scale, const StepRotation& ro, int pos) {
-    if (!ro.cos_t) { rows_of(x, p, rg, scale); return; }
+__device__ __forceinline__ void rotated_rows_of(float4 (&x)[NR / 4], const TA* p, int rg, float scale, const StepRotation& ro, int pos, int vec) {
+    if (!ro.cos_t && !vec) { rows_of(x, p, rg, scale); return; }
     const int half = ro.rot >> 1;
+    if (vec) {
+#pragma unroll
+        for (int m = 0; m < NR / 4; ++m) {
+            const int i = rg * NR + 4 * m;
+            x[m] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i >= DK) continue;
+            float4 own = ld4(p + i);
+            if (ro.cos_t && i < ro.rot) {
+                const bool first = i < half;
+                const float4 other = ld4(p + (first ? i + half : i - half));
+                const float4 c = ld4(ro.cos_t + (size_t)pos * half + (first ? i : i - half));
+                float4 s = ld4(ro.sin_t + (size_t)pos * half + (first ? i : i - half));
+                if (first) s = scaled(s, -1.f);
+                own = make_float4(own.x * c.x + other.x * s.x, own.y * c.y + other.y * s.y, own.z * c.z + other.z * s.z,
+                                  own.w * c.w + other.w * s.w);
+            }
+            x[m] = scaled(own, scale);
+        }
+        return;
+    }
 #pragma unroll
     for (int m = 0; m < NR / 4; ++m) {
         float e[4];
@@ -1090,7 +1111,7 @@ __global__ void __launch_bounds__(WORKERS)
 head_step_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ k, int k_stride, const TA* __restrict__ v,
                  int v_stride, const float* __restrict__ decay, int a_stride, const float* __restrict__ gain, int g_stride,
                  float q_scale, float* __restrict__ out, float* __restrict__ state, const int* __restrict__ cu_q,
-                 const int* __restrict__ state_slots, int H, int dv, int share, StepRotation ro) {
+                 const int* __restrict__ state_slots, int H, int dv, int share, StepRotation ro, int vec) {
     pdl_trigger();
     pdl_wait();
     const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS;
@@ -1107,8 +1128,8 @@ head_step_kernel(const TA* __restrict__ q, int q_stride, const TA* __restrict__ 
     const float a = decay[(size_t)t * a_stride + h], g = gain ? gain[(size_t)t * g_stride + h] : 1.f;
     const int pos = ro.cos_t ? ro.positions[t] : 0;
     float4 kk[NR / 4], qq[NR / 4];
-    rotated_rows_of(kk, k + (size_t)t * k_stride + (size_t)kh * DK, rg, 1.f, ro, pos);
-    rotated_rows_of(qq, q + (size_t)t * q_stride + (size_t)kh * DK, rg, q_scale, ro, pos);
+    rotated_rows_of(kk, k + (size_t)t * k_stride + (size_t)kh * DK, rg, 1.f, ro, pos, vec);
+    rotated_rows_of(qq, q + (size_t)t * q_stride + (size_t)kh * DK, rg, q_scale, ro, pos, vec);
 #pragma unroll
     for (int j = 0; j < C; ++j) {
         float vj = ok[j] ? to_f32<TA>(v[(size_t)t * v_stride + (size_t)h * dv + c0 + cg * C + j]) : 0.f;
@@ -1209,10 +1230,11 @@ RI_API int ri_head_scan(const void* q, int q_stride, const void* k, int k_stride
     const bool narrow = 2 * ctas <= ri_device_sms();
     const int vec = DK % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && aligned4(q, esize) && aligned4(k, esize);
     const StepRotation ro{positions, cos_t, sin_t, rot, interleaved};
+    const int step_vec = vec && (!cos_t || (!interleaved && rot % 8 == 0 && aligned4(cos_t, 4) && aligned4(sin_t, 4)));
 #define RI_HS(TA) do { \
     if (single) { \
         RI_CHECKED(ri_launch(head_step_kernel<TA>, grid, dim3(WORKERS), 0, s, (const TA*)q, q_stride, (const TA*)k, k_stride, \
-            (const TA*)v, v_stride, decay, a_stride, gain, g_stride, q_scale, out, state, cu_q, state_slots, H, dv, share, ro)); \
+            (const TA*)v, v_stride, decay, a_stride, gain, g_stride, q_scale, out, state, cu_q, state_slots, H, dv, share, ro, step_vec)); \
         break; \
     } \
     static bool allowed = false; \

@@ -52,6 +52,9 @@ def _moe(ff, experts, top, groups=None, shared=None):
 # D: every attention size a multiple of 16, so that the bfloat16 engine's prompt portions run on the tensor-core attention;
 #    eight heads on one kv head, whose single tokens run there too; chunks of 50 (three pages and two tokens); retention
 #    without rotation; all groups kept
+# E: a width and feed-forwards that are no multiple of eight (nothing runs on the tensor cores but what pads), odd sizes
+#    everywhere, a table that ends at 9 positions back, a state-space mixer whose step sizes start at an odd column
+# F: no attention at all: every cache is a state
 CONFIGS = {
     "A": {"architecture": "Dozotar", "width": 96, "vocab": 211, "norm": {"eps": 1e-5}, "layers": [
         dict(_attention(4, 2, 24, 40, 3, 0.3, 50.0, 20), mlp={"kind": "dense", "ff": 136}),
@@ -69,8 +72,17 @@ CONFIGS = {
         dict(_retention(2, 64, 48, [0.999, 0.95]), mlp=_moe(32, 8, 2, (4, 1))),
         dict(_attention(8, 1, 32, 16, 3, 0.3, 64.0, 37), mlp={"kind": "dense", "ff": 64}),
         dict(_mamba(4, 16, 64, 2, 4, 2), mlp=_moe(40, 6, 2, (3, 2), 48))]},
+    "E": {"architecture": "Dozotar", "width": 92, "vocab": 101, "norm": {"eps": 1e-4}, "layers": [
+        dict(_attention(3, 3, 23, 9, 4, 0.3, 9.0, 21), mlp=_moe(22, 7, 4, None, 13)),
+        dict(_mamba(3, 6, 15, 1, 3, 3), mlp={"kind": "dense", "ff": 30}),
+        dict(_attention(5, 1, 40, 24, 2, 0.2, 77.0, 64), mlp=_moe(26, 6, 1, (6, 1), None)),
+        dict(_retention(3, 14, 10, [0.98, 0.7, 0.999], (6, 50.0)), mlp=_moe(18, 4, 2, (2, 1), 20))]},
+    "F": {"architecture": "Dozotar", "width": 48, "vocab": 80, "norm": {"eps": 1e-5}, "layers": [
+        dict(_mamba(2, 24, 16, 2, 4, 1), mlp=None),
+        dict(_retention(2, 16, 16, [0.95, 0.99], (16, 1000.0)), mlp=_moe(16, 4, 2)),
+        dict(_mamba(3, 16, 20, 1, 2, 3), mlp={"kind": "dense", "ff": 64})]},
 }
-REL_ROWS = {("A", 0): 8, ("B", 1): 16, ("C", 1): 5, ("D", 0): 32, ("D", 2): 12}
+REL_ROWS = {("A", 0): 8, ("B", 1): 16, ("C", 1): 5, ("D", 0): 32, ("D", 2): 12, ("E", 0): 6, ("E", 2): 16}
 
 
 def tensor_shapes(name: str) -> Dict[str, tuple]:
