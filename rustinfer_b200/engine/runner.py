@@ -15,6 +15,7 @@ launched with an index the kernels could not follow.
 """
 from __future__ import annotations
 
+import gc
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Sequence, Tuple
 
@@ -154,8 +155,16 @@ class _DecodeGraph:
         from ..ops import library as _lib
         before = _lib.launch_count
         self.graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(self.graph, pool=runner._graph_pool):
-            self.logits = runner.model.forward(self.step, runner.entry_caches, self.rows)
+        # an engine that was dropped may still hold graphs and events in reference cycles: were the garbage collector to run
+        # during the capture, destroying them would invalidate it
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(self.graph, pool=runner._graph_pool):
+                self.logits = runner.model.forward(self.step, runner.entry_caches, self.rows)
+        finally:
+            if collecting:
+                gc.enable()
         self.kernels_per_replay = _lib.launch_count - before
         if runner._graph_pool is None:
             runner._graph_pool = self.graph.pool()

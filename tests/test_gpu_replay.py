@@ -521,3 +521,32 @@ def test_long_decoding_on_the_tma_fed_attention_with_and_without_dependent_launc
     for key, outs in results.items():
         for a, b in zip(base, outs):
             assert rel_err(b, a) <= TOL["bfloat16"] / 2, key
+
+
+def test_capture_beside_graphs_left_to_the_garbage_collector(models):
+    """A runner that is dropped while it holds captured steps in a reference cycle is not collected in the middle of the next
+    one's capture (with a collection at nearly every allocation outside of it)."""
+    import gc
+    from rustinfer_b200.engine.runner import ModelRunner, StepEntry
+    folder = models[sorted(models)[0]][0]
+
+    def make():
+        r = ModelRunner(folder, dtype="bfloat16", max_model_len=64, page_size=16, num_pages=8, max_batch_seqs=2,
+                        max_batch_tokens=64, capture_sizes=[1, 2])
+        r.open("a")
+        r.step([StepEntry("a", [1, 2, 3], [2])])
+        return r
+    old = make()
+    want = old.step([StepEntry("a", [4], [0])]).clone()
+    old.cycle = old
+    fresh = make()
+    limits = gc.get_threshold()
+    gc.disable()
+    del old
+    gc.set_threshold(1)
+    gc.enable()
+    try:
+        got = fresh.step([StepEntry("a", [4], [0])])
+    finally:
+        gc.set_threshold(*limits)
+    assert fresh.graph_replays == 1 and torch.equal(got, want)
