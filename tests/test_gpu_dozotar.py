@@ -396,7 +396,7 @@ def test_bucket_bias_attention_edges_and_far_keys(dk, dv, H, G, size, rows, far)
 
 
 @pytest.mark.parametrize("T,E,top,d,groups", [(150, 8, 3, 96, (4, 2)), (5, 6, 1, 83, None), (40, 3, 3, 64, None), (300, 40, 5, 64, (8, 3)),
-                                              (64, 12, 3, 128, (3, 2))])
+                                              (64, 15, 4, 128, (5, 3))])
 @pytest.mark.parametrize("gated", [True, False])
 def test_router_softmax_over_all_with_group_maxima(T, E, top, d, groups, gated):
     x, router = rnd(T, d, seed=1), rnd(E + gated, d, seed=2, scale=0.3)
