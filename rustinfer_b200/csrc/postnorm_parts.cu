@@ -128,7 +128,7 @@ __global__ void latent_prepare_kernel(const TI* __restrict__ proj, int row_strid
                                       const float* __restrict__ sin_t, const int* __restrict__ slot_of_token,
                                       TA* __restrict__ cache, TA* __restrict__ q_plain, TA* __restrict__ q_full,
                                       int H, int d, int r, int rank, const TI* __restrict__ low_base, int low_stride,
-                                      int interleaved) {
+                                      int interleaved, int has_low) {
     pdl_trigger();
     pdl_wait();
     __shared__ float red[33];
@@ -152,6 +152,7 @@ __global__ void latent_prepare_kernel(const TI* __restrict__ proj, int row_strid
         o[ia] = from_f32<TA>(u * c - v * s);
         o[ib] = from_f32<TA>(v * c + u * s);
     }
+    if (!has_low) return;                                     // queries over rows that another layer cached
     // the low-rank vector and the shared key part: behind the queries in the same row, or rows of their own
     const TI* low = low_base ? low_base + (size_t)t * low_stride : row + (size_t)H * (d + r);
     float ss = 0.f;
@@ -265,17 +266,18 @@ RI_API int ri_diff_combine(const float* a, float lambda, float out_scale, float 
 // in_dtype: of proj (and low); act_dtype: of q_plain, q_full and the cache; w_dtype: of the low-rank vector's norm weight.
 // low (may be null): rows [rank + r] of `low_stride` elements that hold the low-rank vector and the shared key part
 // where they do not follow the queries in proj's rows.  interleaved: rotary pairs (2i, 2i+1), else (i, i + r/2).
+// has_low 0: proj holds queries only and nothing is cached.
 // The cache of one layer is [pages][page][rank + r]: a token's row lies at slot_of_token[t] * (rank + r).
 RI_API int ri_latent_prepare(const void* proj, int in_dtype, int row_stride, const void* c_w, int w_dtype, float eps,
                              const int* positions, const float* cos_t, const float* sin_t, const int* slot_of_token,
                              void* cache, void* q_plain, void* q_full, int act_dtype, int tokens, int H, int d, int r,
-                             int rank, const void* low, int low_stride, int interleaved, void* stream) {
+                             int rank, const void* low, int low_stride, int interleaved, int has_low, void* stream) {
     if (tokens <= 0) return 0;
     if (r < 0 || (r & 1) || (r > 0 && (!cos_t || !sin_t || !positions))) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
 #define RI_LP(TI, TW, TA) RI_CHECKED(ri_launch(latent_prepare_kernel<TI, TW, TA>, dim3(tokens), dim3(256), 0, s, (const TI*)proj, \
         row_stride, (const TW*)c_w, eps, positions, cos_t, sin_t, slot_of_token, (TA*)cache, (TA*)q_plain, (TA*)q_full, H, d, r, rank, \
-        (const TI*)low, low_stride, interleaved))
+        (const TI*)low, low_stride, interleaved, has_low))
     if (act_dtype == RI_BF16) {
         if (in_dtype == RI_BF16) { if (w_dtype == RI_BF16) RI_LP(bf16, bf16, bf16); else RI_LP(bf16, float, bf16); }
         else { if (w_dtype == RI_BF16) RI_LP(float, bf16, bf16); else RI_LP(float, float, bf16); }

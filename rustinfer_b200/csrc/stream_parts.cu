@@ -168,7 +168,8 @@ __global__ void hyper_collect_kernel(float* __restrict__ X, int fresh, const TY*
 // its own, over one set of values); a page then holds Hkv heads of keys and Hv heads of values.
 // `conv` (w null: none), for a step in which token t is the one token of entry t: every channel first passes a short
 // causal convolution over time, y = sum_j w[c][j] x_(t - taps + 1 + j), whose earlier inputs come from the entry's state
-// slot, which the new input is shifted into (a channel of an entry is one thread's work).
+// slot, which the new input is shifted into (a channel of an entry is one thread's work).  `q_scale` (null: none) [positions]:
+// the token's queries are multiplied by q_scale[its position] before they are rounded.
 struct QkvConv {
     const float* w;              // [channels][taps]
     float* state;                // [slots][taps - 1][channels], oldest first
@@ -200,7 +201,7 @@ __global__ void __launch_bounds__(1024) qkv_prepare_kernel(const TI* __restrict_
                                    const float* __restrict__ sin_t, int rot, int interleaved,
                                    const int* __restrict__ slot_of_token, TA* __restrict__ cache,
                                    TA* __restrict__ q_out, int Hq, int Hkv, int Hv, int dk, int dv, int has_kv, int page_size,
-                                   QkvConv cv) {
+                                   QkvConv cv, const float* __restrict__ q_scale) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float sm[];
@@ -256,7 +257,8 @@ __global__ void __launch_bounds__(1024) qkv_prepare_kernel(const TI* __restrict_
         }
         __syncthreads();
     }
-    for (int i = tid; i < nq; i += nth) q_out[(size_t)t * nq + i] = from_f32<TA>(qs[i]);
+    const float qf = q_scale ? q_scale[positions[t]] : 1.f;
+    for (int i = tid; i < nq; i += nth) q_out[(size_t)t * nq + i] = from_f32<TA>(qs[i] * qf);
     const int slot = has_kv && cache && slot_of_token ? slot_of_token[t] : -1;
     if (slot < 0) {
         if (cv.w)                                             // the values' inputs are state all the same
@@ -330,14 +332,15 @@ RI_API int ri_hyper_collect(float* X, int fresh, const void* y, int y_dtype, con
 }
 
 // in_dtype: of qkv; act_dtype: of q_out and the cache; w_dtype: of the norm weights.  bias is fp32.  conv_w (may be null):
-// see QkvConv.
+// see QkvConv.  q_scale (may be null): fp32 by position.
 RI_API int ri_qkv_prepare(const void* qkv, int in_dtype, int row_stride, const float* bias, const void* q_w,
                           const void* k_w, int w_dtype, int norm_mode, float eps, const int* positions,
                           const float* cos_t, const float* sin_t, int rot, int interleaved, const int* slot_of_token,
                           void* cache, void* q_out, int act_dtype, int tokens, int Hq, int Hkv, int dk, int dv,
                           int has_kv, int page_size, int value_heads, const float* conv_w, float* conv_state,
-                          const int* conv_slots, int conv_taps, void* stream) {
+                          const int* conv_slots, int conv_taps, const float* q_scale, void* stream) {
     if (tokens <= 0) return 0;
+    if (q_scale && !positions) return (int)cudaErrorInvalidValue;
     if (conv_w && (!conv_slots || conv_taps < 1 || conv_taps > 8 || (conv_taps > 1 && !conv_state))) return (int)cudaErrorInvalidValue;
     const QkvConv cv{conv_w, conv_state, conv_slots, conv_taps};
     // with the convolution a step has few tokens and a thread waits for its channel's state: more threads a token
@@ -355,7 +358,7 @@ RI_API int ri_qkv_prepare(const void* qkv, int in_dtype, int row_stride, const f
             configured = true; } \
         RI_CHECKED(ri_launch(qkv_prepare_kernel<TI, TA, TW>, dim3(tokens), dim3(threads), smem, s, (const TI*)qkv, row_stride, bias, \
             (const TW*)q_w, (const TW*)k_w, norm_mode, eps, positions, cos_t, sin_t, rot, interleaved, slot_of_token, (TA*)cache, \
-            (TA*)q_out, Hq, Hkv, Hv, dk, dv, has_kv, page_size, cv)); } while (0)
+            (TA*)q_out, Hq, Hkv, Hv, dk, dv, has_kv, page_size, cv, q_scale)); } while (0)
     if (act_dtype == RI_BF16) {
         if (in_dtype == RI_BF16) { if (w_dtype == RI_BF16) RI_QP(bf16, bf16, bf16); else RI_QP(bf16, bf16, float); }
         else { if (w_dtype == RI_BF16) RI_QP(float, bf16, bf16); else RI_QP(float, bf16, float); }

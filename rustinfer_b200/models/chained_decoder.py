@@ -170,7 +170,7 @@ class ChainedDecoder:
     def forward(self, step: StepContext, caches: List, logit_rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
         d, T, sms = self.d, step.num_tokens, self.ctx.num_sms
         h = self.h[:T]
-        d.embed.forward(step, h)
+        d.embed.forward(step, h, *d.stem_cache(caches))
         chains = self._chains(T, step, caches)
         K.decode_chain(chains[0][0], chains[0][1], T, sms)
         for i, (block, _) in enumerate(self.entries):

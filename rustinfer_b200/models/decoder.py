@@ -10,7 +10,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..parts import (attention, attention_variants, experts, ffn, hyper, linear_attention, norm, parallel,  # noqa: F401
-                     recurrent_unit, rope, short_conv, state_space, stem_tail)  # (registers the built-in parts)
+                     recurrent_unit, rope, short_conv, state_space, stem_tail, token_input)  # (registers the built-in parts)
 from ..parts.base import EMBEDDINGS, HEADS, NORMS, BuildContext, CacheNeed, ParamDecl, StepContext, StepIndex
 from ..parts.block import Block, Hidden
 from ..parts.spec import ModelSpec
@@ -54,14 +54,18 @@ class Decoder:
         return decls
 
     def cache_needs(self) -> List[Tuple[int, Optional[CacheNeed], Optional[int]]]:
-        """Per run entry: (layer, what its mixer keeps between steps, entry whose cache it reads)."""
-        return [(e.layer, self.blocks[e.layer].mixer.cache_need(), e.cache_of) for e in self.spec.run_order]
+        """Per run entry: (layer, what its mixer keeps between steps, entry whose cache it reads).  A stem that keeps
+        something is one entry more, behind the layers' (layer -1)."""
+        needs = [(e.layer, self.blocks[e.layer].mixer.cache_need(), e.cache_of) for e in self.spec.run_order]
+        if self.embed.cache_need() is not None:
+            needs.append((-1, self.embed.cache_need(), None))
+        return needs
 
     def step_indices(self) -> List[StepIndex]:
         """The index arrays the model's parts want made for every step, each key once."""
         seen: Dict = {}
         for b in self.blocks:
-            for part in (b.mixer, b.ffn):
+            for part in (b.mixer, b.ffn, b.side):
                 if part is None:
                     continue
                 for need in part.step_indices():
@@ -99,29 +103,34 @@ class Decoder:
         self.chained = ChainedDecoder.build(self)
 
     # --------------------------------------------------------------------------- run
+    def stem_cache(self, caches: List) -> Tuple:
+        """The cache of a stem that keeps something (it lies behind the layers'), as the rest of its arguments."""
+        return (caches[len(self.spec.run_order)],) if self.embed.cache_need() is not None else ()
+
     def forward(self, step: StepContext, caches: List, logit_rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
         """Run the tokens of `step`; returns fp32 logits [rows, vocab] at `logit_rows`
         (token indices, int32, device), or None when no logits are wanted."""
         s = self.spec
+        stem = self.stem_cache(caches)
         if self.chained is not None and self.chained.takes(step):
             return self.chained.forward(step, caches, logit_rows)
         if s.streams:
             # several residual streams, all equal to the embedding's output at first: only the first is
             # written until a sublayer's output has been mixed in
             h = torch.empty((s.streams, step.num_tokens, s.hidden_size), dtype=torch.float32, device=self.ctx.device)
-            self.embed.forward(step, h[0])
+            self.embed.forward(step, h[0], *stem)
             hidden = Hidden(h, None, fresh=True)
         elif s.depth_average:
             # every run entry's result is kept beside the stem's output; the layers hand on averages of them
             hist = torch.empty((len(s.run_order) + 1, step.num_tokens, s.hidden_size), dtype=torch.float32,
                                device=self.ctx.device)
-            self.embed.forward(step, hist[0])
+            self.embed.forward(step, hist[0], *stem)
             hidden = Hidden(hist[0], None, history=hist, depth=1,
                             average=torch.empty((step.num_tokens, s.hidden_size), dtype=torch.float32,
                                                 device=self.ctx.device))
         else:
             h = torch.empty((step.num_tokens, s.hidden_size), dtype=torch.float32, device=self.ctx.device)
-            self.embed.forward(step, h)
+            self.embed.forward(step, h, *stem)
             hidden = Hidden(h, None)
         for i, e in enumerate(s.run_order):
             self.blocks[e.layer].forward(hidden, step, caches[i])

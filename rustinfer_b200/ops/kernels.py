@@ -923,7 +923,8 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight: Optio
                 slot_of_token: Optional[torch.Tensor], cache: Optional[torch.Tensor], q_out: torch.Tensor,
                 num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, has_kv: bool,
                 value_heads: Optional[int] = None,
-                conv: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None) -> None:
+                conv: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None,
+                q_scale: Optional[torch.Tensor] = None) -> None:
     """qkv [T, Hq*hd (+ Hkv*hd + Hkv*vd when `has_kv`)]: add `bias` (fp32), norm q and k (`norm_mode` 0: not;
     1: every head by its own root mean square, weights [hd]; 2: all heads at once, weights [Hq*hd] and
     [Hkv*hd]), rotate the first `rotary_dim` channels of every head (pairs (2i, 2i+1) when `interleaved`, else
@@ -932,8 +933,11 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight: Optio
     heads: kv heads times the attention maps of a head).  qkv may be the leading columns of wider rows.  `conv`
     (weight fp32 [columns, taps], state fp32 [slots, taps - 1, columns], state_slots int32 [T]), for a step in which
     row t is the one token of entry t: every column first passes the short convolution as `short_conv` computes it,
-    its earlier inputs from state[state_slots[t]], which the new input is shifted into."""
-    require_cuda(qkv, bias, q_weight, k_weight, positions, cos, sin, slot_of_token, cache, q_out, *(conv or ()))
+    its earlier inputs from state[state_slots[t]], which the new input is shifted into.  `q_scale` (fp32 [positions]):
+    q is multiplied by q_scale[position] before it is rounded."""
+    require_cuda(qkv, bias, q_weight, k_weight, positions, cos, sin, slot_of_token, cache, q_out, q_scale, *(conv or ()))
+    if q_scale is not None and (q_scale.dtype != torch.float32 or q_scale.dim() != 1 or not q_scale.is_contiguous()):
+        raise KernelError("qkv_prepare: q_scale is fp32 [positions]")
     _i32(positions, "positions"); _i32(slot_of_token, "slot_of_token")
     T = qkv.shape[0]
     Hv = value_heads or num_kv_heads
@@ -976,7 +980,7 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight: Optio
                                   dtype_code(ws[0].dtype) if ws else 0, int(norm_mode), float(eps), _p(positions),
                                   _p(cos), _p(sin), int(rotary_dim), 1 if interleaved else 0, _p(slot_of_token), _p(cache),
                                   _p(q_out), dtype_code(q_out.dtype), T, num_heads, num_kv_heads, head_dim, value_dim,
-                                  1 if has_kv else 0, page, Hv, _p(cw), _p(cs), _p(cslots), int(taps), stream_ptr()), "qkv_prepare")
+                                  1 if has_kv else 0, page, Hv, _p(cw), _p(cs), _p(cslots), int(taps), _p(q_scale), stream_ptr()), "qkv_prepare")
 
 
 # ------------------------------------------------------------------------ routed experts
@@ -1380,6 +1384,43 @@ def part_norm_gate(o: torch.Tensor, z: torch.Tensor, weight: Optional[torch.Tens
                                      dtype_code(out.dtype), T, int(parts), n // int(parts), stream_ptr()), "part_norm_gate")
 
 
+# ------------------------------------------------------------ parts that look token ids up in tables
+def embed_pairs(ids: torch.Tensor, positions: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, entries: int,
+                last_token: torch.Tensor, table: torch.Tensor, scale: float, pairs: torch.Tensor, mul_prev: int, mul_cur: int,
+                out: torch.Tensor) -> None:
+    """out[t, :] (fp32) = scale * table[ids[t], :] + pairs[row, :], row = (previous id * mul_prev + id * mul_cur) mod buckets,
+    or `buckets` at position 0; pairs is [buckets + 1, d].  The id before an entry's first token is last_token[slot] (int32,
+    one element a slot), where the entry's last id is left.  `entries`: how many cu_q and state_slots describe."""
+    require_cuda(ids, positions, cu_q, state_slots, last_token, table, pairs, out)
+    for t, n in ((ids, "ids"), (positions, "positions"), (cu_q, "cu_q"), (state_slots, "state_slots"), (last_token, "last_token")):
+        _i32(t, n)
+    T, d = ids.numel(), table.shape[1]
+    _contig(table, "table"); _contig(pairs, "pairs"); _contig(out, "out"); _contig(last_token, "last_token")
+    if out.dtype != torch.float32 or out.shape != (T, d) or pairs.shape[1] != d or pairs.shape[0] < 2:
+        raise KernelError(f"embed_pairs: out is fp32 [{T}, {d}], pairs [buckets + 1, {d}]")
+    if positions.numel() < T or cu_q.numel() < entries + 1 or state_slots.numel() < entries or not 1 <= entries <= T:
+        raise KernelError("embed_pairs: positions [T], cu_q [entries + 1], state_slots [entries]")
+    buckets, most = pairs.shape[0] - 1, (1 << 62) // max(1, table.shape[0])
+    if not (0 <= mul_prev <= most and 0 <= mul_cur <= most):
+        raise KernelError("embed_pairs: the factors are not negative and their products with two ids fit 64 bits")
+    check(L.core().ri_embed_pairs(_p(ids), _p(positions), _p(cu_q), int(entries), _p(state_slots), _p(last_token), _p(table),
+                                  dtype_code(table.dtype), float(scale), _p(pairs), dtype_code(pairs.dtype), int(mul_prev), int(mul_cur),
+                                  buckets, _p(out), T, d, table.shape[0], stream_ptr()), "embed_pairs")
+
+
+def token_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, column: int, out: torch.Tensor) -> None:
+    """out[t, j] = gelu_tanh(z[t, j]) * table[ids[t], column + j]: z fp32 [T, n] (may be a column view), table [vocab, columns]."""
+    require_cuda(z, ids, table, out)
+    _i32(ids, "ids"); _contig(table, "table"); _contig(out, "out")
+    T, n = z.shape
+    if z.dtype != torch.float32 or z.stride(1) != 1 or out.shape != z.shape or ids.numel() < T:
+        raise KernelError("token_gate: z is fp32 [T, n] with unit column stride, out has its shape, ids [T]")
+    if not 0 <= column <= table.shape[1] - n:
+        raise KernelError("token_gate: the columns lie inside the table")
+    check(L.core().ri_token_gate(_p(z), z.stride(0), _p(ids), _p(table), dtype_code(table.dtype), table.shape[1], int(column),
+                                 table.shape[0], _p(out), dtype_code(out.dtype), T, n, stream_ptr()), "token_gate")
+
+
 # ------------------------------------------------- blocks that norm after the sum, and their mixers
 def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Tensor) -> None:
     """out[t,:] (fp32) = scale * table[ids[t],:]."""
@@ -1454,7 +1495,7 @@ def diff_combine(a: torch.Tensor, lam: float, out_scale: float, eps: float, gate
                                    num_heads, value_dim, stream_ptr()), "diff_combine")
 
 
-def latent_prepare(proj: torch.Tensor, c_weight: torch.Tensor, eps: float, positions: torch.Tensor,
+def latent_prepare(proj: torch.Tensor, c_weight: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
                    cos: torch.Tensor, sin: torch.Tensor, slot_of_token: Optional[torch.Tensor],
                    cache: Optional[torch.Tensor], q_plain: torch.Tensor, q_full: torch.Tensor, num_heads: int,
                    head_dim: int, rot_dim: int, rank: int, low: Optional[torch.Tensor] = None,
@@ -1464,19 +1505,23 @@ def latent_prepare(proj: torch.Tensor, c_weight: torch.Tensor, eps: float, posit
     ones into the last r channels of every head of q_full [T, H*(rank+r)], and the cache row of the token
     (the low-rank vector normed with c_weight, then the rotated shared key part) at slot_of_token[t].
     With `low` [T, rank + r] (of proj's dtype, unit column stride) proj holds the queries only, [T, H*(d+r)].
+    With neither `low` nor `c_weight` proj holds the queries only and nothing is cached (the keys are another layer's).
     `interleaved`: the rotary pairs are channels (2i, 2i+1); else (i, i + r/2)."""
     require_cuda(proj, c_weight, positions, cos, sin, slot_of_token, cache, q_plain, q_full, low)
     _i32(positions, "positions"); _i32(slot_of_token, "slot_of_token")
     T, H, d, r = proj.shape[0], num_heads, head_dim, rot_dim
-    cols = H * (d + r) + (0 if low is not None else rank + r)
+    has_low = c_weight is not None
+    if not has_low and (low is not None or cache is not None):
+        raise KernelError("latent_prepare: a cached row needs its norm weight")
+    cols = H * (d + r) + (rank + r if has_low and low is None else 0)
     if proj.stride(1) != 1 or proj.shape[1] != cols:
         raise KernelError(f"latent_prepare: proj is [T, {cols}] with unit column stride")
     if low is not None and (low.dtype != proj.dtype or low.shape != (T, rank + r) or low.stride(1) != 1):
         raise KernelError(f"latent_prepare: low is [T, {rank + r}] of proj's dtype with unit column stride")
-    _contig(q_plain, "q_plain"); _contig(q_full, "q_full"); _contig(c_weight, "c_weight")
+    _contig(q_plain, "q_plain"); _contig(q_full, "q_full")
     if q_plain.shape != (T, H * d) or q_full.shape != (T, H * (rank + r)) or q_plain.dtype != q_full.dtype:
         raise KernelError("latent_prepare: q_plain is [T, H*d], q_full [T, H*(rank+r)], of one dtype")
-    if c_weight.numel() != rank:
+    if has_low and (c_weight.numel() != rank or not c_weight.is_contiguous()):
         raise KernelError("latent_prepare: the norm weight has the low-rank vector's size")
     for t in (cos, sin):
         if t.dtype != torch.float32 or t.shape[1] != r // 2 or not t.is_contiguous():
@@ -1486,10 +1531,10 @@ def latent_prepare(proj: torch.Tensor, c_weight: torch.Tensor, eps: float, posit
         if cache.dtype != q_full.dtype or cache.dim() != 2 or cache.shape[1] % (rank + r):
             raise KernelError("latent_prepare: the cache is [pages, page*(rank+r)] of q's dtype")
     check(L.core().ri_latent_prepare(_p(proj), dtype_code(proj.dtype), proj.stride(0), _p(c_weight),
-                                     dtype_code(c_weight.dtype), float(eps), _p(positions), _p(cos), _p(sin),
+                                     dtype_code(c_weight.dtype) if has_low else 0, float(eps), _p(positions), _p(cos), _p(sin),
                                      _p(slot_of_token), _p(cache), _p(q_plain), _p(q_full), dtype_code(q_full.dtype),
                                      T, H, d, r, rank, _p(low), low.stride(0) if low is not None else 0,
-                                     1 if interleaved else 0, stream_ptr()), "latent_prepare")
+                                     1 if interleaved else 0, 1 if has_low else 0, stream_ptr()), "latent_prepare")
 
 
 def bias_rows(x: torch.Tensor, bias: torch.Tensor) -> None:

@@ -1,11 +1,13 @@
-"""Two more attention mixers over the paged cache, beside `gqa_attention`:
+"""More attention mixers over the paged cache, beside `gqa_attention`:
 
     differential_attention   every head has two softmax maps, with queries and keys of their own, over one
                              set of values; out = rms_head(a1 - lambda a2) * (1 - diff), gated and projected
     latent_attention         keys and values of all heads are made from one cached low-rank vector per token
                              (plus a few rotated key channels the heads share); only that vector is cached
+    distance_bias_attention  (also `gated_attention`) grouped-query attention with the parts such layers share: a bias by
+                             distance or a rotation, a query temperature, a sink, a gate a head
 
-Both run on the fp32-arithmetic attention kernels in both engine precisions: scores, softmax weights and
+All run on the fp32-arithmetic attention kernels in both engine precisions: scores, softmax weights and
 the weighted sum of values are 32-bit there.  The reference engine has one attention
 (crates/infer-worker/src/components/attention.rs:21-37); these are parts of the same kind with caches of
 their own shapes.
@@ -264,7 +266,15 @@ class LatentAttention(Mixer):
         self.rot_layout = str(p.get("rot_layout", "interleaved"))
         if self.rot_layout not in ("half", "interleaved"):
             raise ValueError(f"rot_layout {self.rot_layout!r}: known are 'half' and 'interleaved'")
-        self.gate = bool(p.get("gate", False))
+        self.rot_scaling = dict(p["rot_scaling"]) if p.get("rot_scaling") else None
+        self.gate = {False: "", True: "channel"}.get(p.get("gate") or False, p.get("gate"))
+        if self.gate not in ("", "channel", "head"):
+            raise ValueError(f"gate {self.gate!r}: known are 'channel' and 'head'")
+        self.window = int(p["window"]) if p.get("window") else None
+        self.cache_window = (int(p["cache_window"]) if p.get("cache_window") else None) if "cache_window" in p else self.window
+        if self.cache_window is not None and (self.window is None or self.cache_window < self.window):
+            raise ValueError(f"the cache keeps {self.cache_window} rows, the mask wants {self.window or 'all'}")
+        self.own_kv = bool(p.get("own_kv", True))
         self.tensor_names = dict(p.get("tensor_names") or {})
         self.kd = self.rank + self.rd                       # a cached row
         if self.rd % 2 or self.rd < 0:
@@ -278,9 +288,11 @@ class LatentAttention(Mixer):
     def param_decls(self) -> Dict[str, ParamDecl]:
         n = self._name
         nq = self.H * (self.hd + self.rd)
-        d = {n("dkv"): ParamDecl((self.kd, self.hidden)), n("dkv.norm"): ParamDecl((self.rank,), init="ones"),
-             n("uk"): ParamDecl((self.H * self.hd, self.rank)), n("uv"): ParamDecl((self.H * self.vd, self.rank)),
+        d = {n("uk"): ParamDecl((self.H * self.hd, self.rank)), n("uv"): ParamDecl((self.H * self.vd, self.rank)),
              n("o"): ParamDecl((self.hidden, self.H * self.vd))}
+        if self.own_kv:
+            d[n("dkv")] = ParamDecl((self.kd, self.hidden))
+            d[n("dkv.norm")] = ParamDecl((self.rank,), init="ones")
         if self.q_rank:
             d[n("dq")] = ParamDecl((self.q_rank, self.hidden))
             d[n("dq.norm")] = ParamDecl((self.q_rank,), init="ones")
@@ -288,19 +300,19 @@ class LatentAttention(Mixer):
         else:
             d[n("q")] = ParamDecl((nq, self.hidden))
         if self.gate:
-            d[n("g")] = ParamDecl((self.H * self.vd, self.hidden))
+            d[n("g")] = ParamDecl((self.H if self.gate == "head" else self.H * self.vd, self.hidden))
         if self.sink:
             d[n("sink")] = ParamDecl((self.H,), init="zeros")
         return d
 
     def cache_need(self):
-        return PagedKV(1, self.kd, None, value_dim=self.rank, value_in_key=True)
+        return PagedKV(1, self.kd, self.cache_window, value_dim=self.rank, value_in_key=True)
 
     def prepare(self, ctx: BuildContext) -> None:
         super().prepare(ctx)
-        self.attend = PlainAttend(ctx, self.H, 1, self.kd, self.rank, value_in_key=True)
+        self.attend = PlainAttend(ctx, self.H, 1, self.kd, self.rank, value_in_key=True, window=self.window)
         self.position = shared_position(ctx, PartSpec("rope", {
-            "head_dim": self.rd, "rotary_dim": self.rd, "theta": self.rot_base, "scaling": None,
+            "head_dim": self.rd, "rotary_dim": self.rd, "theta": self.rot_base, "scaling": self.rot_scaling,
             "layout": self.rot_layout})) if self.rd else None
 
     def step_indices(self):
@@ -310,14 +322,15 @@ class LatentAttention(Mixer):
         n = self._name
         # one product for everything that reads the mixer's input: queries (or their low-rank vector), the
         # cached row, the gate
-        parts = [tensors[n("dq") if self.q_rank else n("q")], tensors[n("dkv")]] + ([tensors[n("g")]] if self.gate else [])
+        parts = ([tensors[n("dq") if self.q_rank else n("q")]] + ([tensors[n("dkv")]] if self.own_kv else [])
+                 + ([tensors[n("g")]] if self.gate else []))
         dt = torch.float32 if any(t.dtype == torch.float32 for t in parts) else parts[0].dtype
         self.proj = Linear(torch.cat([t.to(dt) for t in parts], dim=0), self.ctx.num_sms)
         self.uq = self.q_norm = None
         if self.q_rank:
             self.uq = Linear(tensors[n("uq")], self.ctx.num_sms)
             self.q_norm = tensors[n("dq.norm")].to(torch.float32).contiguous()
-        self.c_norm = tensors[n("dkv.norm")].contiguous()
+        self.c_norm = tensors[n("dkv.norm")].contiguous() if self.own_kv else None
         act = self.ctx.dtype
         self.w_uk = tensors[n("uk")].to(act).view(self.H, self.hd, self.rank).contiguous()
         self.w_uv = tensors[n("uv")].to(act).view(self.H, self.vd, self.rank).transpose(1, 2)     # [H, rank, vd]
@@ -334,14 +347,16 @@ class LatentAttention(Mixer):
         q_full = torch.empty((T, H * self.kd), dtype=dt, device=x.device)
         cos, sin = (self.position.cos, self.position.sin) if self.position is not None else (self._no_rot, self._no_rot)
         nq = self.q_rank or H * (self.hd + self.rd)
+        n_low = nq + (self.kd if self.own_kv else 0)          # the gates' first column
+        writes = self.own_kv and cache.writes
         if self.q_rank:
             cq = torch.empty((T, self.q_rank), dtype=dt, device=x.device)
             K.rms_sandwich(proj[:, :nq], None, None, None, self.q_norm, cq, self.norm_eps)
-            queries, low = self.uq(cq, out_dtype=torch.float32), proj[:, nq: nq + self.kd]
+            queries, low = self.uq(cq, out_dtype=torch.float32), proj[:, nq: n_low] if self.own_kv else None
         else:
-            queries, low = proj[:, : nq + self.kd], None
+            queries, low = proj[:, : n_low], None
         K.latent_prepare(queries, self.c_norm, self.norm_eps, step.positions, cos, sin,
-                         g.slot_of_token if cache.writes else None, cache.kv if cache.writes else None,
+                         g.slot_of_token if writes else None, cache.kv if writes else None,
                          q_plain, q_full, H, self.hd, self.rd, self.rank, low=low,
                          interleaved=self.rot_layout == "interleaved")
         # q' of every head into the first kv_rank channels of its row of q_full
@@ -353,7 +368,7 @@ class LatentAttention(Mixer):
         torch.bmm(lat.view(T, H, self.rank).transpose(0, 1), self.w_uv, out=y.view(T, H, self.vd).transpose(0, 1))
         if self.gate:
             gated = torch.empty_like(y)
-            K.sigmoid_gate(y, proj[:, nq + self.kd:], 1, gated)
+            K.sigmoid_gate(y, proj[:, n_low:], self.vd if self.gate == "head" else 1, gated)
             y = gated
         return self.o(y, out_dtype=torch.float32)
 
@@ -379,22 +394,27 @@ def bucket_bias(table: torch.Tensor, far: float, reach: Optional[int] = None) ->
     return table.to(torch.float32)[index].t().contiguous()
 
 
+@register_mixer("gated_attention")
 @register_mixer("distance_bias_attention")
 class DistanceBiasAttention(Mixer):
-    """Grouped-query attention without rotation, whose scores carry a distance bias:
+    """Grouped-query attention whose scores may carry a distance bias:
 
         score(i, j) = q_i . k_j * scale - slope_h * (i - j),    slope_h = 2^(-slope_exponent * (h + 1) / H)
         or            q_i . k_j * scale + rel[bucket(i - j), h]   (`bias` "buckets"; see `distance_bucket`)
+        or            q_i . k_j * scale                           (`bias` "none")
 
     for head h of H, over the keys of a sliding window (None: every earlier key) and of the query's own block of `block`
     positions (None: no blocks).  params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim, scale, window, block,
-    bias ("slopes", the default, or "buckets" with bias_far, the distance of the last row), slope_exponent (default 8),
-    conv_taps (None; else q, k and v pass a short causal convolution a channel right after their projection, weights
+    bias ("slopes", the default, "buckets" with bias_far, the distance of the last row, or "none"), slope_exponent (default 8),
+    proj_bias (q, k and v have biases `q.b` and so on, added in the projection), conv_taps (None; else q, k and v pass a short
+    causal convolution a channel right after their projection, weights
     `q.conv` [channels, taps] and so on), qk_norm_eps (None; else one RMS norm over all heads of q and one over all of k,
-    weights `q.norm`, `k.norm` of those sizes, after the convolution), sink (the softmax's denominator
+    weights `q.norm`, `k.norm` of those sizes, after the convolution), position (PartSpec of a rotary encoding of q and k, or
+    None), q_temperature (PartSpec of a `query_temperature`, or None: q is multiplied by its factor), sink (the softmax's
+    denominator
     holds exp(sink_h), a learned number per head with no key or value), head_gate (head h's output is multiplied
     by sigmoid of the h-th of H numbers W_g x), tensor_names.  Tensors: q, k, v, o, and `sink` [H], `g` [H, hidden], `rel`
-    [rows, H] where asked for; no biases.  With a convolution the caches are (pages, the convolution's inputs); it and the
+    [rows, H] where asked for.  With a convolution the caches are (pages, the convolution's inputs); it and the
     norm run in the launch that writes the cache when every entry brings one token.  q, k, v and the gates are one product of the input; scores, softmax weights and
     their product with the values are fp32 in both engines (the kernels `PlainAttend` picks).  Beside another mixer
     (`parallel_mixers`) it takes the joint product's columns as `proj`, and with a gate a head an `out_scale` on what
@@ -412,8 +432,11 @@ class DistanceBiasAttention(Mixer):
         self.window = int(p["window"]) if p.get("window") else None
         self.block = int(p["block"]) if p.get("block") else None
         self.bias = str(p.get("bias", "slopes"))
-        if self.bias not in ("slopes", "buckets"):
-            raise ValueError(f"distance bias {self.bias!r}: known are 'slopes' and 'buckets'")
+        if self.bias not in ("slopes", "buckets", "none"):
+            raise ValueError(f"distance bias {self.bias!r}: known are 'slopes', 'buckets' and 'none'")
+        self.proj_bias = bool(p.get("proj_bias", False))
+        self.position_spec: Optional[PartSpec] = p.get("position")
+        self.temperature_spec: Optional[PartSpec] = p.get("q_temperature")
         self.bias_far = float(p["bias_far"]) if self.bias == "buckets" else 0.0
         self.qk_norm_eps = float(p["qk_norm_eps"]) if p.get("qk_norm_eps") is not None else None
         self.slope_exponent = float(p.get("slope_exponent", 8.0))
@@ -442,6 +465,9 @@ class DistanceBiasAttention(Mixer):
             d[n("g")] = ParamDecl((self.H, self.hidden))
         if self.bias == "buckets":
             d[n("rel")] = ParamDecl((-1, self.H))
+        if self.proj_bias:
+            for x, size in (("q", self.nq), ("k", self.nk), ("v", self.nv)):
+                d[n(x + ".b")] = ParamDecl((size,), init="zeros")
         if self.qk_norm_eps is not None:
             d[n("q.norm")] = ParamDecl((self.nq,), init="ones")
             d[n("k.norm")] = ParamDecl((self.nk,), init="ones")
@@ -457,6 +483,8 @@ class DistanceBiasAttention(Mixer):
     def prepare(self, ctx: BuildContext) -> None:
         super().prepare(ctx)
         self.attend = PlainAttend(ctx, self.H, self.G, self.hd, self.vd, window=self.window, block=self.block)
+        self.position = shared_position(ctx, self.position_spec)
+        self.temperature = shared_position(ctx, self.temperature_spec)
         self.slopes = None
         if self.bias != "slopes":
             return
@@ -473,7 +501,9 @@ class DistanceBiasAttention(Mixer):
         self.proj = Linear(torch.cat([t.to(dt) for t in parts], dim=0), self.ctx.num_sms)
         self.o = Linear(tensors[n("o")], self.ctx.num_sms)
         self.sink_values = tensors[n("sink")].to(torch.float32).contiguous() if self.sink else None
-        self.bias_rows = self.q_norm = self.k_norm = None
+        self.bias_rows = self.q_norm = self.k_norm = self.qkv_bias = None
+        if self.proj_bias:
+            self.qkv_bias = torch.cat([tensors[n(x + ".b")].to(torch.float32) for x in ("q", "k", "v")]).contiguous()
         if self.bias == "buckets":
             reach = min([r for r in (self.window, self.block) if r], default=None)
             self.bias_rows = bucket_bias(tensors[n("rel")], self.bias_far, reach)
@@ -493,16 +523,20 @@ class DistanceBiasAttention(Mixer):
             proj = self.proj(x, out_dtype=torch.float32)
         nqkv = self.nq + self.nk + self.nv
         q = torch.empty((T, self.nq), dtype=dt, device=x.device)
-        qkv, conv = proj[:, :nqkv], None
+        qkv, conv, qkv_bias = proj[:, :nqkv], None, self.qkv_bias
         if conv_cache is not None:
             if step.max_q_len == 1 and step.num_entries == T:
                 conv = (self.conv.weight, conv_cache.state, step.state_slots)
             else:
                 qkv = self.conv.run(qkv, step, conv_cache, torch.empty((T, nqkv), dtype=torch.float32, device=x.device),
-                                    residual=False)
-        K.qkv_prepare(qkv, None, self.q_norm, self.k_norm, 0 if self.qk_norm_eps is None else 2, self.qk_norm_eps or 0.0,
-                      step.positions, None, None, 0, False, g.slot_of_token if cache.writes else None,
-                      cache.kv if cache.writes else None, q, self.H, self.G, self.hd, self.vd, True, conv=conv)
+                                    residual=False, in_bias=qkv_bias)
+                qkv_bias = None                               # it stands in front of the convolution
+        pos = self.position
+        K.qkv_prepare(qkv, qkv_bias, self.q_norm, self.k_norm, 0 if self.qk_norm_eps is None else 2, self.qk_norm_eps or 0.0,
+                      step.positions, pos.cos if pos else None, pos.sin if pos else None, pos.rotary_dim if pos else 0,
+                      bool(pos and pos.layout == "interleaved"), g.slot_of_token if cache.writes else None,
+                      cache.kv if cache.writes else None, q, self.H, self.G, self.hd, self.vd, True, conv=conv,
+                      q_scale=self.temperature.factor if self.temperature else None)
         if self.head_gate:
             o = torch.empty((T, self.H * self.vd), dtype=torch.float32, device=x.device)
             self.attend(q, o, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes,

@@ -5,7 +5,8 @@ model around it.  It declares the tensors it owns (`param_decls`), receives them
 (`load`), and runs on what the step hands it.  New kinds are added by registering a
 class; no file of the framework changes.
 
-    Embedding      forward(step, h_fp32[T,hidden]) fills the stream for the step's tokens (the stem)
+    Embedding      forward(step, h_fp32[T,hidden]) fills the stream for the step's tokens (the stem); one that
+                   keeps something between steps (cache_need()) gets its cache as a third argument
     Mixer          forward(x[T,hidden], step, cache) -> delta[T,hidden]
                    cache_need() -> PagedKV | FixedState | None
                    step_indices() -> the int32 arrays it wants made for every step
@@ -257,8 +258,12 @@ def shared_position(ctx: BuildContext, spec: Optional[PartSpec]) -> Optional[Any
 class Embedding(Part):
     """The stem: turns the step's token ids (and, if it wants, positions) into the fp32 stream."""
 
-    def forward(self, step: StepContext, h: torch.Tensor) -> None:
-        """Fill h [step.num_tokens, hidden] (fp32)."""
+    def cache_need(self) -> Optional["FixedState"]:
+        """State of fixed size the stem keeps of every request (earlier token ids, say), or None."""
+        return None
+
+    def forward(self, step: StepContext, h: torch.Tensor, cache: Optional["StateLayerCache"] = None) -> None:
+        """Fill h [step.num_tokens, hidden] (fp32).  `cache` is given to a stem that has a `cache_need` only."""
         raise NotImplementedError
 
     def shared_table(self) -> Optional[torch.Tensor]:

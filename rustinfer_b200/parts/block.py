@@ -39,6 +39,7 @@ class Block:
         self.mixer_norm: Optional[Norm] = NORMS.build(spec.mixer_norm) if spec.mixer_norm else None
         self.ffn: Optional[FeedForward] = FEED_FORWARDS.build(spec.ffn) if spec.ffn else None
         self.ffn_norm: Optional[Norm] = NORMS.build(spec.ffn_norm) if spec.ffn_norm else None
+        self.side: Optional[FeedForward] = FEED_FORWARDS.build(spec.side) if spec.side else None
         self.extra_norms: Dict[str, Norm] = {role: NORMS.build(ps) for role, ps in spec.extra_norms.items()}
         fn = ARRANGEMENTS.get(spec.arrangement)
         if fn is None:
@@ -50,7 +51,8 @@ class Block:
 
     def roles(self):
         """role -> part, for every part the layer has."""
-        named = {"mixer": self.mixer, "mixer_norm": self.mixer_norm, "ffn": self.ffn, "ffn_norm": self.ffn_norm}
+        named = {"mixer": self.mixer, "mixer_norm": self.mixer_norm, "ffn": self.ffn, "ffn_norm": self.ffn_norm,
+                 "side": self.side}
         named.update(self.extra_norms)
         return {role: part for role, part in named.items() if part is not None}
 
@@ -60,7 +62,7 @@ class Block:
 
     @property
     def graph_safe(self) -> bool:
-        return self.mixer.graph_safe and (self.ffn is None or self.ffn.graph_safe)
+        return all(part is None or part.graph_safe for part in (self.mixer, self.ffn, self.side))
 
     def forward(self, hidden: Hidden, step: StepContext, cache) -> None:
         self._run(self, hidden, step, cache)
@@ -87,24 +89,31 @@ def _pre_norm(block: Block, hidden: Hidden, step: StepContext, cache) -> None:
 def _sandwich(block: Block, hidden: Hidden, step: StepContext, cache) -> None:
     """A norm before and a norm after each sublayer:
 
-        h += post_mixer_norm(mixer(mixer_norm(h)));  h += post_ffn_norm(ffn(ffn_norm(h)))
+        h += post_mixer_norm(mixer(mixer_norm(h)));  h += post_ffn_norm(ffn(ffn_norm(h)));  h += post_side_norm(side(h))
 
-    (the second line only when the layer has a feed-forward).  The norms after the sublayers go
-    by the roles `post_mixer_norm` and `post_ffn_norm` in `extra_norms`.  A sublayer's output stays
-    pending as a `NormedDelta`; the next norm that reads the stream, of this layer, the next or
-    the model's last, norms it, adds it and norms the sum in one kernel."""
+    (the second only when the layer has a feed-forward, the third only when it has a `side` part, which reads the
+    stream itself, rounded to the activation dtype).  The norms after the sublayers go by the roles `post_mixer_norm`,
+    `post_ffn_norm` and `post_side_norm` in `extra_norms`.  A sublayer's output stays pending as a `NormedDelta`; the next
+    norm that reads the stream, of this layer, the next or the model's last, norms it, adds it and norms the sum in one
+    kernel.  In front of a side part the pending output is normed and added, and the sum rounded, in one kernel (its norm
+    is an `rmsnorm`)."""
     from .norm import NormedDelta
     post_mixer, post_ffn = block.extra_norms.get("post_mixer_norm"), block.extra_norms.get("post_ffn_norm")
     if block.mixer_norm is None or post_mixer is None:
         raise ValueError("the sandwich arrangement wants a norm before and a norm after the mixer")
     x = block.mixer_norm.add_norm(hidden.stream, hidden.pending)
     hidden.pending = NormedDelta(block.mixer.forward(x, step, cache), post_mixer)
-    if block.ffn is None:
-        return
-    if block.ffn_norm is None or post_ffn is None:
-        raise ValueError("the sandwich arrangement wants a norm before and a norm after the feed-forward")
-    x = block.ffn_norm.add_norm(hidden.stream, hidden.pending)
-    hidden.pending = NormedDelta(block.ffn.forward(x, step), post_ffn)
+    if block.ffn is not None:
+        if block.ffn_norm is None or post_ffn is None:
+            raise ValueError("the sandwich arrangement wants a norm before and a norm after the feed-forward")
+        x = block.ffn_norm.add_norm(hidden.stream, hidden.pending)
+        hidden.pending = NormedDelta(block.ffn.forward(x, step), post_ffn)
+    if block.side is not None:
+        post_side = block.extra_norms.get("post_side_norm")
+        if post_side is None:
+            raise ValueError("the sandwich arrangement wants a norm after the side part")
+        x = hidden.pending.norm.add_output(hidden.stream, hidden.pending.delta)
+        hidden.pending = NormedDelta(block.side.forward(x, step), post_side)
 
 
 def _hyper(block: Block, hidden: Hidden, step: StepContext, cache) -> None:
@@ -204,6 +213,19 @@ def settle_depth(hidden: Hidden) -> torch.Tensor:
         hidden.pending.run(None, None)
         hidden.pending = None
     return hidden.stream
+
+
+def settled_stream(hidden: Hidden) -> torch.Tensor:
+    """A copy of the stream with what the last sublayer left pending (a tensor or a `NormedDelta`) added, for inspection;
+    nothing of `hidden` is changed."""
+    from ..ops import kernels as K
+    from .norm import NormedDelta
+    h = hidden.stream.clone()
+    if isinstance(hidden.pending, NormedDelta):
+        hidden.pending.norm.add_into(h, hidden.pending.delta)
+    elif hidden.pending is not None:
+        K.residual_add(h, hidden.pending)
+    return h
 
 
 def _sandwich_depth_average(block: Block, hidden: Hidden, step: StepContext, cache) -> None:

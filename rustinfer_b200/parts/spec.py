@@ -46,8 +46,10 @@ class LayerSpec:
     mixer_norm: Optional[PartSpec] = None
     ffn: Optional[PartSpec] = None
     ffn_norm: Optional[PartSpec] = None
-    names: Mapping[str, str] = field(default_factory=dict)   # role -> prefix; roles: mixer, mixer_norm, ffn, ffn_norm, extras
+    names: Mapping[str, str] = field(default_factory=dict)   # role -> prefix; roles: mixer, mixer_norm, ffn, ffn_norm, side, extras
     arrangement: str = "pre_norm"
+    # a third sublayer behind the feed-forward (a registered feed-forward kind) in arrangements that run one
+    side: Optional[PartSpec] = None
     extra_norms: Mapping[str, PartSpec] = field(default_factory=dict)   # role -> norm
 
 

@@ -15,7 +15,7 @@ from typing import Dict, Optional
 import torch
 
 from ..ops import kernels as K
-from .base import Embedding, Head, ParamDecl, StepContext, register_embedding, register_head
+from .base import Embedding, FixedState, Head, ParamDecl, StateLayerCache, StepContext, register_embedding, register_head
 from .linear import Linear
 
 
@@ -60,6 +60,38 @@ class ScaledEmbedding(TokenEmbedding):
 
     def forward(self, step: StepContext, h: torch.Tensor) -> None:
         K.embed_scaled(step.token_ids[: step.num_tokens], self.table, self.scale, h)
+
+
+@register_embedding("bigram_embedding")
+class BigramEmbedding(ScaledEmbedding):
+    """h[t, :] = scale * E[ids[t], :] + P[row, :], with row = (ids[t-1] * mul_prev + ids[t] * mul_cur) mod buckets, and the
+    table's last row, `buckets`, for the first token of a request; sum and product in fp32.  The token before an entry's first
+    one is state of the request (one int32 a slot).  params: as `scaled_embedding`, buckets, mul_prev, mul_cur, bigram_name
+    (local name of P [buckets + 1, hidden], default "bigram")."""
+
+    def __init__(self, params):
+        super().__init__(params)
+        self.buckets = int(params["buckets"])
+        self.mul_prev, self.mul_cur = int(params["mul_prev"]), int(params["mul_cur"])
+        self.bigram_name = str(params.get("bigram_name", "bigram"))
+        if self.buckets <= 0 or min(self.mul_prev, self.mul_cur) < 0:
+            raise ValueError("bigram_embedding: buckets is positive, the factors are not negative")
+        self.pairs: Optional[torch.Tensor] = None
+
+    def param_decls(self) -> Dict[str, ParamDecl]:
+        return {**super().param_decls(), self.bigram_name: ParamDecl((self.buckets + 1, self.hidden))}
+
+    def cache_need(self) -> FixedState:
+        return FixedState((1,), "int32")
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        super().load(tensors)
+        self.pairs = tensors[self.bigram_name].contiguous()
+
+    def forward(self, step: StepContext, h: torch.Tensor, cache: StateLayerCache) -> None:
+        n = step.num_tokens
+        K.embed_pairs(step.token_ids[:n], step.positions[:n], step.cu_q, step.state_slots, step.num_entries, cache.state,
+                      self.table, self.scale, self.pairs, self.mul_prev, self.mul_cur, h)
 
 
 @register_embedding("sinusoid_embedding")
