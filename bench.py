@@ -17,7 +17,7 @@ attention), the Llama-3.2-3B-shaped model at 8 of its 28 layers serving 64 reque
 this engine's attention and GEMM kernels timed against the reference's own attention kernels
 (compiled unmodified, see baseline/reference_kernels.py) and the library GEMM on the same data.
 `--shape` takes the layer sizes of the 3B or 8B benchmark configuration for the headline instead;
-`--only decode|prefill|serve` runs one part alone and prints its time.  `--family dirurax` (or `pikalix`, `sotazen`, `linedra`, `dozotar`) leaves
+`--only decode|prefill|serve` runs one part alone and prints its time.  `--family dirurax` (or `pikalix`, `sotazen`, `linedra`, `dozotar`, `fotulix`) leaves
 all of that aside and prints a line of its own: prefill and decode of that family's models at two sizes beside
 Llama models of the same width, depth, feed-forward width and vocabulary, and that family's kernels alone against
 their rooflines.
@@ -909,24 +909,17 @@ def sotazen_kernels(hbm_gbs, bf16_tflops, size):
         q = bf(B, Hq * hd)
         o = torch.empty(B, Hq * vd, device=dev, dtype=torch.float32 if maps > 1 else torch.bfloat16)
         span = min(ctx, window) if window else ctx
-        if att.fast_single:
-            ranges, kernel = att._splits(B, ctx), "one CTA a key head"
-            us = time_kernel(lambda: K.attention_single(q, o, cache, table, cu, kv_len, ent, Hq, Hkv, hd, hd ** -0.5, window, None, vd,
-                                                        sink=sink_values is not None, splits=ranges, part=att.part, softcap=softcap,
-                                                        sink_values=sink_values, maps=maps, value_in_key=vik), flush=flush)
-        elif att.rows_single:
-            ranges, kernel = att._rows_splits(B, ctx), "tensor cores, 64 (token, head) rows a CTA"
-            us = time_kernel(lambda: K.attention_rows(q, o, cache, table, cu, kv_len, ent, att.zero_tok0[:B], Hq, Hkv, hd, hd ** -0.5,
-                                                      window, vd, sink=sink_values is not None, softcap=softcap,
-                                                      sink_values=sink_values, maps=maps, value_in_key=vik, splits=ranges,
-                                                      part=att.part), flush=flush)
+        if att.fast_single or att.rows:
+            ranges = att.ranges(B, ctx)
+            kernel = "one CTA a key head" if att.fast_single else "tensor cores, 16 heads a CTA"
+            us = time_kernel(lambda: att.single_tokens(q, o, cache, table, cu, kv_len, ent, ctx, hd ** -0.5, sink=sink_values is not None,
+                                                       softcap=softcap, sink_values=sink_values), flush=flush)
         else:
             ranges, t0 = 0, i32([0] * B)
-            fn, kernel = ((K.attention_rows, "tensor cores, 64 (token, head) rows a CTA") if att.rows else
-                          (lambda *a, **k: K.attention_plain(*a[:13], None, *a[13:], **k), "fp32 arithmetic, 16 rows a head"))
-            us = time_kernel(lambda: fn(q, o, cache, table, cu, kv_len, ent, t0, Hq, Hkv, hd, hd ** -0.5, window, vd,
-                                        sink=sink_values is not None, softcap=softcap, sink_values=sink_values,
-                                        maps=maps, value_in_key=vik), repeats=5, flush=flush)
+            kernel = "fp32 arithmetic, 16 rows a head"
+            us = time_kernel(lambda: K.attention_plain(q, o, cache, table, cu, kv_len, ent, t0, Hq, Hkv, hd, hd ** -0.5, window, None, vd,
+                                                       sink=sink_values is not None, softcap=softcap, sink_values=sink_values,
+                                                       maps=maps, value_in_key=vik), repeats=5, flush=flush)
         return {"us": round(us, 1), "ranges": ranges, "hbm_frac": frac(B * span * per * 2, us), "kernel": kernel,
                 "useful_tflops": round(2 * B * span * Hq * (hd + vd) / (us * 1e-6) / 1e12, 2)}
     res = single(2 * ah, akv, ad, av, 2, False, win, 50.0, None)
@@ -1117,15 +1110,9 @@ def linedra_kernels(hbm_gbs, bf16_tflops, size):
     q, o = bf(B, ah * ad), torch.empty(B, ah * av, device=dev)
     res = {}
     for name, sl in (("us", slopes), ("no_bias_us", None)):
-        if att.fast_single:
-            ranges = att._splits(B, ctx)
-            us = time_kernel(lambda: K.attention_single(q, o, cache, table, cu, kv_len, ent, ah, akv, ad, ad ** -0.5, win, None, av,
-                                                        sink=True, splits=ranges, part=att.part, sink_values=sink, slopes=sl), flush=flush)
-        else:
-            ranges = att._rows_splits(B, ctx) if att.rows_single else 1
-            us = time_kernel(lambda: K.attention_rows(q, o, cache, table, cu, kv_len, ent, att.zero_tok0[:B] if att.rows_single else i32([0] * B),
-                                                      ah, akv, ad, ad ** -0.5, win, av, sink=True, sink_values=sink, splits=ranges,
-                                                      part=att.part, slopes=sl), flush=flush)
+        ranges = att.ranges(B, ctx)
+        us = time_kernel(lambda: att.single_tokens(q, o, cache, table, cu, kv_len, ent, ctx, ad ** -0.5, sink=True, sink_values=sink,
+                                                   slopes=sl), flush=flush)
         res[name] = round(us, 1)
     res.update(ranges=ranges, hbm_frac=frac(B * min(ctx, win) * per * 2, res["us"]),
                no_bias_hbm_frac=frac(B * min(ctx, win) * per * 2, res["no_bias_us"]))
@@ -1324,9 +1311,8 @@ def dozotar_kernels(hbm_gbs, bf16_tflops, size):
     att = PlainAttend(bctx, ah, akv, ad, av, block=chunk)
     cache = bf(B * nblk, 2, akv, PAGE, ad)
     q, o = bf(B, ah * ad), torch.empty(B, ah * av, device=dev, dtype=torch.bfloat16)
-    ranges = att._splits(B, ctx)
-    run = lambda bi: timed(lambda: K.attention_single(q, o, cache, table, cu, kv_len, ent, ah, akv, ad, ad ** -0.5, None, chunk, av,
-                                                      splits=ranges, part=att.part, bias=bi))
+    ranges = att.ranges(B, ctx)
+    run = lambda bi: timed(lambda: att.single_tokens(q, o, cache, table, cu, kv_len, ent, ctx, ad ** -0.5, bias=bi))
     moved = B * chunk * akv * (ad + av) * 2
     entry("bucket_attention_decode64", run(bias), moved, [("no_bias", run(None), moved)], ranges=ranges)
     T = 2048
@@ -1357,8 +1343,209 @@ def dozotar_kernels(hbm_gbs, bf16_tflops, size):
     return out
 
 
+def _fotulix(width, layers, ff, vocab, attn, rotary, latent, window, side, buckets):
+    """`layers` layers in the order attention, latent attention (rows of its own), attention, latent attention (that one's
+    rows), attention, rotated attention, attention, latent attention (the same rows); a dense feed-forward and an input by
+    token in each."""
+    ah, akv, ad, av = attn
+    rh, rkv, rd, rv = rotary
+    th, td, tr, tv, rank = latent
+    out = []
+    for i in range(layers):
+        if i % 2 == 0:
+            layer = {"type": "attention", "mixer": {"heads": ah, "kv_heads": akv, "dim": ad, "vdim": av, "scale": ad ** -0.5,
+                                                    "bias_max": 128, "q_temp": {"coef": 0.1, "every": 1024}}}
+        elif i % 8 == 5:
+            layer = {"type": "attention_2", "mixer": {"heads": rh, "kv_heads": rkv, "dim": rd, "vdim": rv, "scale": rd ** -0.5, "rot": {
+                "dims": rd // 2, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+        else:
+            mixer = {"heads": th, "dim": td, "rot_dim": tr, "vdim": tv, "kv_rank": rank, "scale": (td + tr) ** -0.5,
+                     "mask": {"size": window}, "rot": {"dims": tr, "base": 10000.0, "scaling": {
+                         "factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+            if i > 1:
+                mixer["kv_from"] = 1
+            layer = {"type": "latent_attention", "mixer": mixer}
+        out.append(dict(layer, mlp={"kind": "dense", "ff": ff}))
+    return {"architecture": "Fotulix", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "embedding": {"scale": 1.0, "bigram": {"buckets": buckets, "mul_prev": 40503, "mul_cur": 9973}}, "token_side": {"dim": side},
+            "layers": out}
+
+
+# Fotulix at the same widths: attention with the bias (heads, kv heads, key, value), rotated attention with a sink, latent
+# attention as Sotazen's (heads, plain, rotated, value, rank) under the other families' window, channels of the input by token
+FOTULIX_SIZES = {
+    "w1024": dict(width=1024, layers=8, ff=4096, vocab=32768, attn=(16, 4, 64, 64), rotary=(8, 2, 128, 128), latent=(16, 64, 32, 64, 128),
+                  window=1024, side=128, buckets=65521, llama=(16, 4, 64)),
+    "w2048": dict(width=2048, layers=8, ff=8192, vocab=32768, attn=(32, 8, 64, 64), rotary=(16, 4, 128, 128), latent=(32, 64, 32, 64, 256),
+                  window=1024, side=256, buckets=65521, llama=(32, 8, 64)),
+}
+
+
+def fotulix_kernels(hbm_gbs, bf16_tflops, size):
+    """The Fotulix kernels alone at one size, each beside the like kernel of the nearest existing family on the same
+    shapes (the scaled embedding, Linedra's norms around a sublayer, the q, k, v and latent preparations without the
+    new options, the attentions without bias, rotation's sink or window, Pikalix's attention in a prompt): microseconds, and
+    what that is of the bytes they must move at the measured copy bandwidth."""
+    import torch
+    from rustinfer_b200.ops import kernels as K
+    from rustinfer_b200.parts.attention_variants import PlainAttend, bucket_bias
+    from rustinfer_b200.parts.base import BuildContext
+    dev = torch.device("cuda:0")
+    sz = FOTULIX_SIZES[size]
+    d = sz["width"]
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    bf = lambda *s: torch.randn(*s, device=dev).to(torch.bfloat16)
+    f32 = lambda *s: torch.randn(*s, device=dev)
+    frac = lambda moved, us: round(moved / (us * 1e-6) / 1e9 / hbm_gbs, 4)
+    timed = lambda fn: time_kernel(fn, flush=flush)
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+    out = {}
+
+    def entry(name, us, moved, likes=(), **more):
+        r = {"us": round(us, 1), "hbm_frac": frac(moved, us)}
+        for like, lus, lmoved in likes:
+            r[like + "_us"], r[like + "_hbm_frac"] = round(lus, 1), frac(lmoved, lus)
+        r.update(more)
+        out[name] = r
+    ah, akv, ad, av = sz["attn"]
+    rh, rkv, rd, rv = sz["rotary"]
+    th, td, tr, tv, rank = sz["latent"]
+    kd, win, side, vocab, layers = rank + tr, sz["window"], sz["side"], sz["vocab"], sz["layers"]
+    table, pairs, stable = bf(vocab, d), bf(sz["buckets"] + 1, d), bf(vocab, side * layers)
+    for tag, T, entries in (("prefill2048", 2048, 1), ("decode64", 64, 64)):
+        cu = i32([i * (T // entries) for i in range(entries + 1)])
+        slots = i32(list(range(entries)))
+        ids = torch.randint(0, vocab, (T,), device=dev, dtype=torch.int32)
+        pos = i32(list(range(T)))
+        last = torch.zeros(entries + 1, 1, dtype=torch.int32, device=dev)
+        h = torch.empty(T, d, device=dev)
+        entry(f"embed_pairs_{tag}", timed(lambda: K.embed_pairs(ids, pos, cu, slots, entries, last, table, 1.0, pairs, 40503, 9973, h)),
+              T * d * (2 + 2 + 4), [("embed_scaled", timed(lambda: K.embed_scaled(ids, table, 1.0, h)), T * d * (2 + 4))])
+        # the norm of a sublayer's output, the add and the rounded copy beside the norms around a sublayer
+        y, w = f32(T, d), f32(d)
+        xo = torch.empty(T, d, device=dev, dtype=torch.bfloat16)
+        entry(f"norm_add_{tag}", timed(lambda: K.norm_add(h, y, w, 1e-6, xo)), T * d * (4 + 4 + 4 + 2), [
+            ("rms_sandwich", timed(lambda: K.rms_sandwich(h, y, w, h, w, xo, 1e-6)), T * d * (4 + 4 + 4 + 2))])
+        # the input by token: gate product, gate by token, projection (all of the part), beside the feed-forward's two products
+        wg, wp = bf(side, d), bf(d, side)
+        z, g, so = torch.empty(T, side, device=dev), torch.empty(T, side, device=dev, dtype=torch.bfloat16), torch.empty(T, d, device=dev)
+        x16 = bf(T, d)
+        K.gemm_tc(x16, wg, z, K.EPI_F32)
+        zs = f32(T, side)
+        entry(f"token_gate_{tag}", timed(lambda: K.token_gate(z, ids, stable, side, g)), T * side * (4 + 2 + 2), [
+            ("sigmoid_gate", timed(lambda: K.sigmoid_gate(zs, zs, 1, g)), T * side * (4 + 4 + 2))])
+
+        def part():
+            K.gemm_tc(x16, wg, z, K.EPI_F32)
+            K.token_gate(z, ids, stable, side, g)
+            K.gemm_tc(g, wp, so, K.EPI_F32)
+        wgu, wdn = bf(2 * side, d), bf(d, side)
+        m = torch.empty(T, side, device=dev, dtype=torch.bfloat16)
+
+        def ffn():
+            K.gemm_tc(x16, wgu, m, K.EPI_SILU)
+            K.gemm_tc(m, wdn, so, K.EPI_F32)
+        moved = 2 * d * side * 2 + T * d * (2 + 4)
+        entry(f"token_input_{tag}", timed(part), moved, [("gated_ffn_same_width", timed(ffn), moved + d * side * 2)])
+        # q, k, v: biases and the temperature; rotation
+        sl = i32(list(range(T)))
+        fac, cos, sin = f32(4096), f32(4096, rd // 4), f32(4096, rd // 4)
+        qc = ah * ad + akv * (ad + av)
+        qkv, qb = f32(T, qc + ah), f32(qc)
+        cache = bf(T // PAGE + 1, 2, akv, PAGE, ad)
+        qo = torch.empty(T, ah * ad, device=dev, dtype=torch.bfloat16)
+        prep = lambda b, f: K.qkv_prepare(qkv[:, :qc], b, None, None, 0, 0.0, pos, None, None, 0, False, sl, cache, qo, ah, akv, ad, av, True,
+                                          q_scale=f)
+        entry(f"bias_temperature_cache_{tag}", timed(lambda: prep(qb, fac)), T * qc * (4 + 2), [
+            ("without", timed(lambda: prep(None, None)), T * qc * (4 + 2))])
+        rc = rh * rd + rkv * (rd + rv)
+        rqkv, rcache = f32(T, rc + rh), bf(T // PAGE + 1, 2, rkv, PAGE, rd)
+        ro = torch.empty(T, rh * rd, device=dev, dtype=torch.bfloat16)
+        lh, lkv, lhd = sz["llama"]
+        lcols = (lh + 2 * lkv) * lhd
+        l16, lcache, lc = bf(T, lcols), bf(T // PAGE + 1, 2, lkv, PAGE, lhd), f32(4096, lhd // 2)
+        us_rope = timed(lambda: K.rope_scatter(l16, pos, lc, lc, sl, lcache, lh, lkv, lhd, lhd))
+        entry(f"rotate_cache_{tag}", timed(lambda: K.qkv_prepare(rqkv[:, :rc], None, None, None, 0, 0.0, pos, cos, sin, rd // 2, True, sl, rcache,
+                                                                 ro, rh, rkv, rd, rv, True)), T * rc * (4 + 2),
+              [("rope_scatter", us_rope, T * lcols * (2 + 2))])
+        # latent attention: queries over another layer's rows, beside queries and a row of their own
+        nq = th * (td + tr)
+        proj, cw, c3 = f32(T, nq + kd + th), bf(rank), f32(4096, tr // 2)
+        lat = bf(T // PAGE + 1, PAGE * kd)
+        qp, qf = torch.empty(T, th * td, device=dev, dtype=torch.bfloat16), torch.empty(T, th * kd, device=dev, dtype=torch.bfloat16)
+        own = timed(lambda: K.latent_prepare(proj[:, : nq + kd], cw, 1e-6, pos, c3, c3, sl, lat, qp, qf, th, td, tr, rank))
+        entry(f"latent_queries_{tag}", timed(lambda: K.latent_prepare(proj[:, :nq], None, 1e-6, pos, c3, c3, None, None, qp, qf, th, td, tr, rank)),
+              T * nq * (4 + 2), [("latent_prepare", own, T * (nq + kd) * (4 + 2))])
+    # attentions of 64 single tokens at 4,096 keys, as the parts launch them
+    B, ctx = 64, 4096
+    nblk = ctx // PAGE
+    bctx = BuildContext(dev, torch.bfloat16, ctx, PAGE, max_batch_seqs=B, num_sms=sms)
+    kv_len, cu, ent = i32([ctx] * B), i32(list(range(B + 1))), i32(list(range(B)))
+    btable = torch.randperm(B * nblk, device=dev).to(torch.int32).view(B, nblk).contiguous()
+    bias = bucket_bias(f32(32, ah), 128)
+
+    def single(H, G, hd, vd, vik=False, window=None, fp32_kernel=False, **opts):
+        att = PlainAttend(bctx, H, G, hd, vd, value_in_key=vik, window=window)
+        per = G * (hd + (0 if vik else vd))
+        c = bf(B * nblk, PAGE * per) if vik or hd != vd else bf(B * nblk, 2, G, PAGE, hd)
+        q, o = bf(B, H * hd), torch.empty(B, H * vd, device=dev, dtype=torch.bfloat16)
+        args = (q, o, c, btable, cu, kv_len, ent)
+        if fp32_kernel:
+            splits = max(1, min(4 * sms // (B * G), 16))
+            part = torch.empty(K.attention_single_scratch_floats(B, H, vd, splits), device=dev)
+            us = timed(lambda: K.attention_single(*args, H, G, hd, hd ** -0.5, window, None, vd, splits=splits, part=part, **opts))
+        else:
+            us = timed(lambda: att.single_tokens(*args, ctx, hd ** -0.5, **opts))
+        return us, B * min(ctx, window or ctx) * per * 2
+    gate, rgate, tgate = f32(B, ah), f32(B, rh), f32(B, th)
+    us, moved = single(ah, akv, ad, av, bias=bias, gate=gate)
+    entry("bias_attention_decode64", us, moved, [("no_bias", *single(ah, akv, ad, av)),
+                                                 ("fp32_arithmetic_kernel", *single(ah, akv, ad, av, bias=bias, fp32_kernel=True))])
+    sink = f32(rh)
+    us, moved = single(rh, rkv, rd, rv, sink=True, sink_values=sink, gate=rgate)
+    entry("sink_attention_decode64", us, moved, [("no_sink", *single(rh, rkv, rd, rv)),
+                                                 ("fp32_arithmetic_kernel", *single(rh, rkv, rd, rv, sink=True, sink_values=sink, fp32_kernel=True))])
+    us, moved = single(th, 1, kd, rank, True, win, gate=tgate)
+    entry("window_latent_attention_decode64", us, moved, [("every_key", *single(th, 1, kd, rank, True))])
+    # a prompt of 2,048 tokens
+    T = 2048
+    tbl, cup, kvl = i32([list(range(T // PAGE))]), i32([0, T]), i32([T])
+
+    def prompt(H, G, hd, vd, vik=False, window=None, **opts):
+        per = G * (hd + (0 if vik else vd))
+        c = bf(T // PAGE, PAGE * per) if vik or hd != vd else bf(T // PAGE, 2, G, PAGE, hd)
+        q, o = bf(T, H * hd), torch.empty(T, H * vd, device=dev, dtype=torch.bfloat16)
+        tl = list(range(0, T, K.attention_rows_tokens_per_tile(H, G, hd, vd)))
+        te, t0 = i32([0] * len(tl)), i32(tl)
+        us = timed(lambda: K.attention_rows(q, o, c, tbl, cup, kvl, te, t0, H, G, hd, hd ** -0.5, window, vd, value_in_key=vik, **opts))
+        n = sum(min(p + 1, window) if window else p + 1 for p in range(T))
+        return round(us, 1), round(2 * n * H * (hd + vd) / (us * 1e-6) / 1e12, 2)
+
+    def like(H, G, hd, window=None):
+        c, q = bf(T // PAGE, 2, G, PAGE, hd), bf(T, H * hd)
+        o = torch.empty(T, H * hd, device=dev, dtype=torch.bfloat16)
+        tl = list(range(0, T, K.mma_tokens_per_tile(H, G)))
+        te, t0 = i32([0] * len(tl)), i32(tl)
+        us = timed(lambda: K.attention_prefill_bf16(q, o, c, tbl, cup, kvl, te, t0, H, G, hd, hd ** -0.5, window, None, precise=True, sink=True))
+        n = sum(min(p + 1, window) if window else p + 1 for p in range(T))
+        return round(us, 1), round(4 * n * H * hd / (us * 1e-6) / 1e12, 2)
+    for name, own, others in (
+            ("bias_attention", lambda: prompt(ah, akv, ad, av, bias=bias, gate=f32(T, ah)),
+             {"no_bias": lambda: prompt(ah, akv, ad, av), "pikalix_kernel": lambda: like(ah, akv, ad)}),
+            ("sink_attention", lambda: prompt(rh, rkv, rd, rv, sink=True, sink_values=sink, gate=f32(T, rh)),
+             {"no_sink": lambda: prompt(rh, rkv, rd, rv), "pikalix_kernel": lambda: like(rh, rkv, rd)}),
+            ("window_latent_attention", lambda: prompt(th, 1, kd, rank, True, win, gate=f32(T, th)), {"every_key": lambda: prompt(th, 1, kd, rank, True)})):
+        us, tf = own()
+        res = {"us": us, "useful_tflops": tf}
+        for k, fn in others.items():
+            res[k + "_us"], res[k + "_useful_tflops"] = fn()
+        out[name + "_prefill2048"] = res
+    return out
+
+
 def family_bench(args) -> int:
-    """`--family dirurax|pikalix|sotazen|linedra|dozotar`: prefill and decode throughput of that family's models at a few sizes beside
+    """`--family dirurax|pikalix|sotazen|linedra|dozotar|fotulix`: prefill and decode throughput of that family's models at a few sizes beside
     Llama models of the same width, depth, feed-forward width and vocabulary (random weights), and the
     family's own kernels alone.  One JSON line."""
     import torch
@@ -1371,7 +1558,8 @@ def family_bench(args) -> int:
     say = lambda msg: print(f"[bench] {msg}", file=sys.stderr, flush=True)
     ctx, tokens = min(args.context, 4096), max(2, min(args.prompt_tokens, 8192))
     family = args.family
-    table = {"pikalix": PIKALIX_SIZES, "sotazen": SOTAZEN_SIZES, "linedra": LINEDRA_SIZES, "dozotar": DOZOTAR_SIZES}.get(family, FAMILY_SIZES)
+    table = {"pikalix": PIKALIX_SIZES, "sotazen": SOTAZEN_SIZES, "linedra": LINEDRA_SIZES, "dozotar": DOZOTAR_SIZES,
+             "fotulix": FOTULIX_SIZES}.get(family, FAMILY_SIZES)
     result = {"family": family, "dtype": "bf16", "data": "synthetic", "peaks": peak_kind, "points": {}, "kernels": {}}
     sizes = [s for s in table if not args.size or s in args.size.split(",")]
     for size in sizes:
@@ -1384,12 +1572,14 @@ def family_bench(args) -> int:
             own = _linedra(**{k: v for k, v in sz.items() if k != "llama"})
         elif family == "dozotar":
             own = _dozotar(**{k: v for k, v in sz.items() if k != "llama"})
+        elif family == "fotulix":
+            own = _fotulix(**{k: v for k, v in sz.items() if k != "llama"})
         else:
             own = _dirurax(sz["width"], sz["layers"], sz["ff"], sz["vocab"], sz["gla"], sz["attn"], sz["delta"], sz["block"])
         configs = {family: own, "llama": _llama_like(sz["width"], sz["layers"], sz["ff"], sz["vocab"], *sz["llama"])}
         if family in ("linedra", "dozotar"):         # also beside the nearest of the other families, at equal size
             configs["pikalix"] = _pikalix(**{k: v for k, v in PIKALIX_SIZES[size].items() if k != "llama"})
-        if family == "dozotar":
+        if family in ("dozotar", "fotulix"):
             configs["sotazen"] = _sotazen(**{k: v for k, v in SOTAZEN_SIZES[size].items() if k != "llama"})
         point = {}
         for fam, cfg in configs.items():
@@ -1426,6 +1616,7 @@ def family_bench(args) -> int:
                                    else sotazen_kernels(hbm_gbs, bf16_tflops, size) if family == "sotazen"
                                    else linedra_kernels(hbm_gbs, bf16_tflops, size) if family == "linedra"
                                    else dozotar_kernels(hbm_gbs, bf16_tflops, size) if family == "dozotar"
+                                   else fotulix_kernels(hbm_gbs, bf16_tflops, size) if family == "fotulix"
                                    else dirurax_kernels(hbm_gbs, size))
         say(f"{size} kernels: {result['kernels'][size]}")
     clocks.stop()
@@ -1460,7 +1651,7 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=CONTEXT, help="with --only: context the decode ends at")
     ap.add_argument("--prompt-tokens", type=int, default=PREFILL_TOKENS,
                     help="with --only prefill: length of the prompt, computed in one step (up to 8192)")
-    ap.add_argument("--family", default="llama", choices=["llama", "dirurax", "pikalix", "sotazen", "linedra", "dozotar"],
+    ap.add_argument("--family", default="llama", choices=["llama", "dirurax", "pikalix", "sotazen", "linedra", "dozotar", "fotulix"],
                     help="dirurax, pikalix: that family's prefill and decode at a few sizes beside Llama models of equal size, "
                          "and its kernels alone (one JSON line of its own; the default workload is unchanged)")
     ap.add_argument("--size", default="", help="with --family dirurax or pikalix: sizes to run, with commas (default: all)")
@@ -1475,7 +1666,7 @@ def main() -> int:
         return 0
     args.warmup = max(args.warmup, 3)
     args.steps = max(args.steps, 2)
-    if args.family in ("dirurax", "pikalix", "sotazen", "linedra", "dozotar"):
+    if args.family in ("dirurax", "pikalix", "sotazen", "linedra", "dozotar", "fotulix"):
         return family_bench(args)
 
     import torch

@@ -49,6 +49,8 @@ constexpr size_t SMEM_FLOATS = (size_t)QT * QS + (size_t)KC * KS + (size_t)KC * 
 //                    query head h, after scale and cap (null: none)
 //   bias             a learned distance bias: bias[h * bias_len + min(query position - key position, bias_len - 1)] is
 //                    added to the score of query head h, after scale and cap (null: none)
+//   gate             head h's output for token t is multiplied by gate_scale * sigmoid(gate[t * gate_stride + h]) before it
+//                    is stored (null: not)
 struct Extra {
     float softcap;
     const float* sink_values;
@@ -57,7 +59,13 @@ struct Extra {
     const float* slopes;
     const float* bias;
     int bias_len;
+    const float* gate;
+    int gate_stride;
+    float gate_scale;
 };
+__device__ __forceinline__ float gate_of(const Extra& ex, int t, int h) {
+    return ex.gate ? ex.gate_scale / (1.0f + expf(-ex.gate[(size_t)t * ex.gate_stride + h])) : 1.f;
+}
 
 // key head and value head of query head h
 __device__ __forceinline__ void heads_of(int h, int Hq, int Hkv, int maps, int& key_head, int& value_head) {
@@ -200,10 +208,11 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ o
     }
     if (row_valid) {
         const float inv = l > 0.f ? 1.0f / l : 0.f;
+        const float den = ex.gate ? 1.0f + expf(-ex.gate[(size_t)(q_begin + j0 + row) * ex.gate_stride + h]) : 1.f;
         TO* o = out + (size_t)(q_begin + j0 + row) * out_stride + (size_t)h * VD + l8;
 #pragma unroll
         for (int i = 0; i < NACC; ++i)
-            if (VD % 8 == 0 || l8 + 8 * i < VD) o[8 * i] = from_f32<TO>(acc[i] * inv);
+            if (VD % 8 == 0 || l8 + 8 * i < VD) o[8 * i] = from_f32<TO>(ex.gate ? ex.gate_scale * (acc[i] * inv) / den : acc[i] * inv);
     }
 }
 
@@ -473,7 +482,8 @@ attention_single_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ 
             dst[d] = total;
             if (d == 0) { dst[VD] = mrun[g]; dst[VD + 1] = l; }
         } else {
-            out[(size_t)t * out_stride + (size_t)(head0 + g * head_step) * VD + d] = from_f32<TO>(l > 0.f ? total / l : 0.f);
+            out[(size_t)t * out_stride + (size_t)(head0 + g * head_step) * VD + d] =
+                from_f32<TO>((l > 0.f ? total / l : 0.f) * gate_of(ex, t, head0 + g * head_step));
         }
     }
 }
@@ -486,7 +496,7 @@ template <typename T>
 __global__ void __launch_bounds__(32)
 attention_single_merge_kernel(const float* __restrict__ part, T* __restrict__ out, int out_stride,
                               const int* __restrict__ cu_q, const int* __restrict__ entry_list,
-                              int Hq, int splits, int sink, const float* __restrict__ sink_values) {
+                              int Hq, int splits, int sink, const float* __restrict__ sink_values, Extra ex) {
     pdl_trigger();
     pdl_wait();
     const int b = entry_list[blockIdx.y], h = blockIdx.x;
@@ -516,7 +526,7 @@ attention_single_merge_kernel(const float* __restrict__ part, T* __restrict__ ou
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
     if (sink) L += expf(sv - M);
-    const float inv = L > 0.f ? 1.f / L : 0.f;
+    const float inv = (L > 0.f ? 1.f / L : 0.f) * gate_of(ex, t, h);
     constexpr int DPL = (VD + 31) / 32;                       // channels a lane
     float acc[DPL];
 #pragma unroll
@@ -579,9 +589,10 @@ RI_API int ri_attention_plain_ex(const void* q, int q_stride, void* out, int out
                                  const int* tile_q0, int n_tiles, int Hq, int Hkv, int page_size,
                                  float scale, int window, int block, int sink, float softcap,
                                  const float* sink_values, int maps, int value_in_key, int out_f32, const float* slopes,
-                                 const float* bias, int bias_len, void* stream) {
+                                 const float* bias, int bias_len, const float* gate, int gate_stride,
+                                 float gate_scale, void* stream) {
     if (n_tiles <= 0) return 0;
-    const Extra ex{softcap, sink_values, maps, value_in_key, slopes, bias, bias_len};
+    const Extra ex{softcap, sink_values, maps, value_in_key, slopes, bias, bias_len, gate, gate_stride, gate_scale};
     if (bias && bias_len <= 0) return (int)cudaErrorInvalidValue;
     if (!extra_fits(Hq, Hkv, ex)) return (int)cudaErrorInvalidValue;
     cudaStream_t s = (cudaStream_t)stream;
@@ -602,7 +613,7 @@ RI_API int ri_attention_plain(const void* q, int q_stride, void* out, int out_st
                               float scale, int window, int block, int sink, void* stream) {
     return ri_attention_plain_ex(q, q_stride, out, out_stride, cache, dtype, block_table, table_stride, cu_q, kv_len,
                                  tile_entry, tile_q0, n_tiles, Hq, Hkv, page_size, scale, window, block, sink,
-                                 0.f, nullptr, 1, 0, 0, nullptr, nullptr, 0, stream);
+                                 0.f, nullptr, 1, 0, 0, nullptr, nullptr, 0, nullptr, 0, 1.f, stream);
 }
 
 // Entries that bring a single token (entry_list[i], -1: skip): keys and values of a kv head are read once
@@ -614,9 +625,10 @@ RI_API int ri_attention_single_ex(const void* q, int q_stride, void* out, int ou
                                   const int* entry_list, int n_entries, int Hq, int Hkv, int page_size, float scale,
                                   int window, int block, int sink, int splits, float* part, float softcap,
                                   const float* sink_values, int maps, int value_in_key, int out_f32,
-                                  const float* slopes, const float* bias, int bias_len, void* stream) {
+                                  const float* slopes, const float* bias, int bias_len, const float* gate, int gate_stride,
+                                 float gate_scale, void* stream) {
     if (n_entries <= 0) return 0;
-    const Extra ex{softcap, sink_values, maps, value_in_key, slopes, bias, bias_len};
+    const Extra ex{softcap, sink_values, maps, value_in_key, slopes, bias, bias_len, gate, gate_stride, gate_scale};
     if (bias && bias_len <= 0) return (int)cudaErrorInvalidValue;
     if (!extra_fits(Hq, Hkv, ex)) return (int)cudaErrorInvalidValue;
     if (Hq / (Hkv * maps) > SG || SV > 4) return (int)cudaErrorNotSupported;
@@ -637,7 +649,7 @@ RI_API int ri_attention_single_ex(const void* q, int q_stride, void* out, int ou
         out_stride, (const T*)cache, block_table, table_stride, cu_q, kv_len, entry_list, Hq, Hkv, page_size, scale, \
         window, block, sink, part, ex)); \
     if (splits > 1) RI_CHECKED(ri_launch(attention_single_merge_kernel<TO>, dim3(Hq, n_entries), dim3(32), 0, s, \
-        (const float*)part, (TO*)out, out_stride, cu_q, entry_list, Hq, splits, sink, sink_values)); } while (0)
+        (const float*)part, (TO*)out, out_stride, cu_q, entry_list, Hq, splits, sink, sink_values, ex)); } while (0)
     if (dtype == RI_BF16 && out_f32) RI_SINGLE(bf16, float);
     else if (dtype == RI_BF16) RI_SINGLE(bf16, bf16);
     else RI_SINGLE(float, float);
@@ -652,7 +664,7 @@ RI_API int ri_attention_single(const void* q, int q_stride, void* out, int out_s
                                int window, int block, int sink, int splits, float* part, void* stream) {
     return ri_attention_single_ex(q, q_stride, out, out_stride, cache, dtype, block_table, table_stride, cu_q, kv_len,
                                   entry_list, n_entries, Hq, Hkv, page_size, scale, window, block, sink, splits, part,
-                                  0.f, nullptr, 1, 0, 0, nullptr, nullptr, 0, stream);
+                                  0.f, nullptr, 1, 0, 0, nullptr, nullptr, 0, nullptr, 0, 1.f, stream);
 }
 
 RI_API int ri_attention_single_supports(int Hq, int Hkv) {

@@ -401,7 +401,8 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, blo
                     scale: float, window: Optional[int], block: Optional[int] = None,
                     value_dim: Optional[int] = None, sink: bool = False, softcap: Optional[float] = None,
                     sink_values: Optional[torch.Tensor] = None, maps: int = 1, value_in_key: bool = False,
-                    slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> None:
+                    slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+                    gate: Optional[torch.Tensor] = None, gate_scale: float = 1.0) -> None:
     """q [T, >=Hq*hd] (may be a column view of the qkv buffer), out [T, Hq*vd].  `block`: a query
     sees only the keys of its own block of that many positions (counted from 0).  `value_dim`:
     size of a value where it is not the keys'; the cache is then [pages, Hkv*page*(hd+vd)].  `sink`:
@@ -413,9 +414,11 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, blo
     its own first `value_dim` channels, and the cache holds keys only.  `slopes` (fp32 [Hq]): a linear
     distance bias, slopes[h] * (query position - key position) taken off head h's scores after scale
     and cap.  `bias` (fp32 [Hq, n]): bias[h, min(query position - key position, n - 1)] added to head h's
-    scores after scale and cap.  `out` may be fp32 whatever the cache's dtype."""
-    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_q0, sink_values, slopes, bias)
+    scores after scale and cap.  `gate` (fp32 [T, Hq], may be a column view): head h's output for token t is multiplied by
+    gate_scale * sigmoid(gate[t, h]) before it is rounded.  `out` may be fp32 whatever the cache's dtype."""
+    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_q0, sink_values, slopes, bias, gate)
     _slopes_ok(slopes, num_heads, bias)
+    _gate_ok(gate, q, num_heads)
     for t, n in ((block_table, "block_table"), (cu_q, "cu_q"), (kv_len, "kv_len"),
                  (tile_entry, "tile_entry"), (tile_q0, "tile_q0")):
         _i32(t, n)
@@ -429,7 +432,7 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, blo
                                     int(window) if window else 0, int(block) if block else 0, 1 if sink else 0,
                                     float(softcap) if softcap else 0.0, _p(sink_values), int(maps),
                                     1 if value_in_key else 0, 1 if out.dtype == torch.float32 else 0, _p(slopes),
-                                    _p(bias), bias.shape[1] if bias is not None else 0, stream_ptr()),
+                                    _p(bias), bias.shape[1] if bias is not None else 0, *_gate_args(gate, gate_scale), stream_ptr()),
           "attention_plain")
 
 
@@ -439,6 +442,15 @@ def _slopes_ok(slopes: Optional[torch.Tensor], num_heads: int, bias: Optional[to
         raise KernelError("attention: bias is contiguous fp32 [heads, distances]")
     if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != num_heads or not slopes.is_contiguous()):
         raise KernelError("attention: slopes is fp32 [heads]")
+
+
+def _gate_ok(gate: Optional[torch.Tensor], q: torch.Tensor, num_heads: int) -> None:
+    if gate is not None and (gate.dtype != torch.float32 or gate.shape != (q.shape[0], num_heads) or gate.stride(1) != 1):
+        raise KernelError("attention: gate is fp32 [tokens, heads] with unit column stride")
+
+
+def _gate_args(gate: Optional[torch.Tensor], gate_scale: float):
+    return _p(gate), gate.stride(0) if gate is not None else 0, float(gate_scale)
 
 
 def _attention_common(q, out, cache, num_heads, num_kv_heads, head_dim, vd, sink_values, maps, value_in_key) -> int:
@@ -469,13 +481,15 @@ def attention_single(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                      block: Optional[int] = None, value_dim: Optional[int] = None, sink: bool = False,
                      splits: int = 1, part: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
                      sink_values: Optional[torch.Tensor] = None, maps: int = 1, value_in_key: bool = False,
-                     slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> None:
+                     slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+                     gate: Optional[torch.Tensor] = None, gate_scale: float = 1.0) -> None:
     """Attention of the entries that bring one token (`entry_list`, int32; -1 skips): fp32 arithmetic, a kv
     head's keys and values read once for all its query heads.  Arguments as `attention_plain`.  `splits` > 1
     cuts every entry's keys into that many ranges, a CTA each, joined by a second launch through `part`
     (fp32, `attention_single_scratch_floats` long)."""
-    require_cuda(q, out, cache, block_table, cu_q, kv_len, entry_list, part, sink_values, slopes, bias)
+    require_cuda(q, out, cache, block_table, cu_q, kv_len, entry_list, part, sink_values, slopes, bias, gate)
     _slopes_ok(slopes, num_heads, bias)
+    _gate_ok(gate, q, num_heads)
     if splits > 1 and (part is None or part.dtype != torch.float32 or not part.is_contiguous() or
                        part.numel() < attention_single_scratch_floats(entry_list.numel(), num_heads, value_dim or head_dim, splits)):
         raise KernelError("attention_single: the scratch for the key ranges is too small")
@@ -491,7 +505,7 @@ def attention_single(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                                      int(splits), _p(part) if splits > 1 else None,
                                      float(softcap) if softcap else 0.0, _p(sink_values), int(maps),
                                      1 if value_in_key else 0, 1 if out.dtype == torch.float32 else 0, _p(slopes),
-                                     _p(bias), bias.shape[1] if bias is not None else 0, stream_ptr()),
+                                     _p(bias), bias.shape[1] if bias is not None else 0, *_gate_args(gate, gate_scale), stream_ptr()),
           "attention_single", 2 if splits > 1 else 1)
 
 
@@ -515,17 +529,43 @@ def attention_rows(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
                    value_dim: Optional[int] = None, sink: bool = False, softcap: Optional[float] = None,
                    sink_values: Optional[torch.Tensor] = None, maps: int = 1, value_in_key: bool = False,
                    splits: int = 1, part: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                   bias: Optional[torch.Tensor] = None, block: Optional[int] = None) -> None:
+                   bias: Optional[torch.Tensor] = None, block: Optional[int] = None,
+                   gate: Optional[torch.Tensor] = None, gate_scale: float = 1.0) -> None:
     """`attention_plain` on the tensor cores for a bf16 cache: the scores are fp32 sums of products of bf16 q and
     k, cap, mask and softmax are fp32, and the softmax weights meet the bf16 values unrounded (three bf16 pieces a
     weight).  Arguments as there; tiles hold `attention_rows_tokens_per_tile` tokens.  `splits` > 1
     cuts every tile's keys into that many ranges, a CTA each, joined by a second launch through `part` (fp32,
     `attention_rows_scratch_floats` long): for few tiles over many keys."""
-    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_tok0, sink_values, part, slopes, bias)
+    _attention_rows("ri_attention_rows", q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_tok0, num_heads,
+                    num_kv_heads, head_dim, scale, window, value_dim, sink, softcap, sink_values, maps, value_in_key, splits, part,
+                    slopes, bias, block, gate, gate_scale)
+
+
+def attention_rows_single(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, cu_q: torch.Tensor,
+                          kv_len: torch.Tensor, entry_list: torch.Tensor, zeros: torch.Tensor, num_heads: int, num_kv_heads: int,
+                          head_dim: int, scale: float, window: Optional[int], value_dim: Optional[int] = None, sink: bool = False,
+                          softcap: Optional[float] = None, sink_values: Optional[torch.Tensor] = None, maps: int = 1,
+                          value_in_key: bool = False, splits: int = 1, part: Optional[torch.Tensor] = None,
+                          slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, block: Optional[int] = None,
+                          gate: Optional[torch.Tensor] = None, gate_scale: float = 1.0) -> None:
+    """`attention_rows` for the entries that bring one token (`entry_list`, int32; -1 skips; `zeros`: at least as many zeros):
+    a CTA's four warps walk the keys of one key head side by side for up to 16 of its query heads.  Arguments as there."""
+    _attention_rows("ri_attention_rows_single", q, out, cache, block_table, cu_q, kv_len, entry_list, zeros, num_heads, num_kv_heads,
+                    head_dim, scale, window, value_dim, sink, softcap, sink_values, maps, value_in_key, splits, part, slopes, bias,
+                    block, gate, gate_scale)
+
+
+def _attention_rows(entry_point, q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_tok0, num_heads, num_kv_heads, head_dim,
+                    scale, window, value_dim, sink, softcap, sink_values, maps, value_in_key, splits, part, slopes, bias, block,
+                    gate, gate_scale) -> None:
+    require_cuda(q, out, cache, block_table, cu_q, kv_len, tile_entry, tile_tok0, sink_values, part, slopes, bias, gate)
     _slopes_ok(slopes, num_heads, bias)
+    _gate_ok(gate, q, num_heads)
     for t, n in ((block_table, "block_table"), (cu_q, "cu_q"), (kv_len, "kv_len"),
                  (tile_entry, "tile_entry"), (tile_tok0, "tile_tok0")):
         _i32(t, n)
+    if tile_tok0.numel() < tile_entry.numel():
+        raise KernelError("attention_rows: a first token for every tile")
     vd = value_dim or head_dim
     if cache.dtype != torch.bfloat16 or q.stride(0) % 8 or q.data_ptr() % 16 or cache.data_ptr() % 16:
         raise KernelError("attention_rows: a bf16 cache and q rows that start on 16-byte boundaries")
@@ -535,19 +575,26 @@ def attention_rows(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
     if splits > 1 and (part is None or part.dtype != torch.float32 or not part.is_contiguous() or part.data_ptr() % 16 or
                        part.numel() < attention_rows_scratch_floats(tile_entry.numel(), num_heads, num_kv_heads, vd, maps, splits)):
         raise KernelError("attention_rows: the scratch for the key ranges is too small")
-    check(L.attention_rows(head_dim, vd).ri_attention_rows(
+    check(getattr(L.attention_rows(head_dim, vd), entry_point)(
         _p(q), q.stride(0), _p(out), out.stride(0), _p(cache), _p(block_table), block_table.stride(0), _p(cu_q),
         _p(kv_len), _p(tile_entry), _p(tile_tok0), tile_entry.numel(), num_heads, num_kv_heads, page_size, float(scale),
         int(window) if window else 0, 1 if sink else 0, float(softcap) if softcap else 0.0, _p(sink_values), int(maps),
         1 if value_in_key else 0, 1 if out.dtype == torch.float32 else 0, int(splits), _p(part) if splits > 1 else None,
-        _p(slopes), _p(bias), bias.shape[1] if bias is not None else 0, int(block) if block else 0, stream_ptr()),
-        "attention_rows", 2 if splits > 1 else 1)
+        _p(slopes), _p(bias), bias.shape[1] if bias is not None else 0, int(block) if block else 0, *_gate_args(gate, gate_scale),
+        stream_ptr()), entry_point[3:], 2 if splits > 1 else 1)
 
 
 def attention_rows_ctas_per_sm(head_dim: int, value_dim: int, value_in_key: bool, out_dtype: torch.dtype) -> int:
     """CTAs of `attention_rows` that one SM holds at once, asked of the driver (at least 1)."""
     n = L.attention_rows(head_dim, value_dim).ri_attention_rows_ctas_per_sm(1 if value_in_key else 0,
                                                                              1 if out_dtype == torch.float32 else 0)
+    return max(1, int(n))
+
+
+def attention_rows_single_ctas_per_sm(head_dim: int, value_dim: int, value_in_key: bool, out_dtype: torch.dtype) -> int:
+    """CTAs of `attention_rows_single` that one SM holds at once, asked of the driver (at least 1)."""
+    n = L.attention_rows(head_dim, value_dim).ri_attention_rows_single_ctas_per_sm(1 if value_in_key else 0,
+                                                                                   1 if out_dtype == torch.float32 else 0)
     return max(1, int(n))
 
 

@@ -30,15 +30,15 @@ from .spec import PartSpec
 
 class PlainAttend:
     """How a mixer sends its queries to the attention kernels with fp32 scores and softmax weights.  The bfloat16
-    engine: prompt portions go to the tensor-core kernel in tiles of 64 (token, head) rows (where the sizes are
-    multiples of 16).  Entries of one token go there too where eight or more query heads share a key head (one
-    cached row for all heads, say: the arithmetic of so many heads a key outgrows the fp32 pipes), else to the
-    kernel that reads a key head once for all its query heads (where it takes the geometry).  Both cut the keys
-    into ranges when few CTAs would walk many keys.  What neither takes runs on the fp32-arithmetic kernel in
-    tiles of 16 query rows.  The 32-bit engine uses that last kernel alone, whose sums do not depend on how the
-    tokens were cut into steps."""
+    engine, where the sizes are multiples of 16: prompt portions go to the tensor-core kernel in tiles of 64 (token, head)
+    rows, entries of one token to its sister for single tokens, whose warps walk the keys of a key head side by side for up to
+    16 of its query heads.  Other sizes: entries of one token go to the fp32-arithmetic kernel that reads a key head once for
+    all its query heads (where it takes the geometry).  All of them cut the keys of single tokens into ranges when few CTAs
+    would walk many keys.  What none of them takes runs on the fp32-arithmetic kernel in tiles of 16 query rows.  The 32-bit
+    engine uses that last kernel alone, whose sums do not depend on how the tokens were cut into steps."""
     MAX_SPLITS = 16             # of the one-CTA-a-key-head kernel
-    ROWS_MAX_SPLITS = 32        # of the tensor-core kernel
+    ROWS_MAX_SPLITS = 32        # of the tensor-core kernel for single tokens
+    MIN_RANGE = 256             # keys of a range, at least: four tiles for every warp
 
     def __init__(self, ctx: BuildContext, heads: int, kv_heads: int, head_dim: int, value_dim: int, maps: int = 1,
                  value_in_key: bool = False, window: Optional[int] = None, block: Optional[int] = None):
@@ -48,8 +48,7 @@ class PlainAttend:
         fast = (ctx.dtype == torch.bfloat16 and os.environ.get("RUSTINFER_B200_BLOCK_ATTENTION", "fast") != "plain")
         self.rows = fast and K.attention_rows_supports(head_dim, value_dim, value_in_key)
         group = heads // (kv_heads * maps)
-        self.rows_single = self.rows and group >= 8
-        self.fast_single = (fast and not self.rows_single
+        self.fast_single = (fast and not self.rows
                             and K.attention_single_supports(heads, kv_heads, head_dim, value_dim, maps))
         rows = K.attention_rows_tokens_per_tile(heads, kv_heads, head_dim, value_dim, maps) if self.rows else 16
         self._single = self.part = None
@@ -60,12 +59,13 @@ class PlainAttend:
                 n = K.attention_single_scratch_floats(ctx.max_batch_seqs, heads, value_dim, self.MAX_SPLITS)
                 ctx.shared[key] = torch.empty(n, dtype=torch.float32, device=ctx.device)
             self.part = ctx.shared[key]
-        elif self.rows_single:
+        elif self.rows:
             self._single = single_token_entries()
-            self.ctas_per_tile = kv_heads * maps * -(-group // 64)
-            # ranges are made until the CTAs fill the SMs once: one CTA more than fit at once costs a second turn
-            self.slots = ctx.num_sms * K.attention_rows_ctas_per_sm(head_dim, value_dim, value_in_key,
-                                                                    torch.float32 if maps > 1 else ctx.dtype)
+            self.ctas_per_entry = kv_heads * maps * -(-group // 16)
+            # ranges are made until there are CTAs for every SM and some more (from there on the join costs more than
+            # the longer walks), and never more than are resident at once
+            self.slots = ctx.num_sms * K.attention_rows_single_ctas_per_sm(head_dim, value_dim, value_in_key,
+                                                                           torch.float32 if maps > 1 else ctx.dtype)
             key = ("rows_scratch", value_dim)
             if key not in ctx.shared or ctx.shared[key].numel() < self.slots * 64 * (value_dim + 2):
                 ctx.shared[key] = torch.empty(self.slots * 64 * (value_dim + 2), dtype=torch.float32, device=ctx.device)
@@ -81,31 +81,39 @@ class PlainAttend:
     def _span(self, max_kv_len: int) -> int:
         return min([max_kv_len] + [n for n in (self.window, self.block) if n])
 
-    def _splits(self, n_single: int, max_kv_len: int) -> int:
-        want = -(-4 * self.ctx.num_sms // max(1, n_single * self.Hkv * self.maps))
-        return max(1, min(want, -(-self._span(max_kv_len) // 128), self.MAX_SPLITS))
+    def ranges(self, n_single: int, max_kv_len: int) -> int:
+        """Ranges the keys of `n_single` single tokens are cut into."""
+        if self.fast_single:
+            want = -(-4 * self.ctx.num_sms // max(1, n_single * self.Hkv * self.maps))
+            return max(1, min(want, -(-self._span(max_kv_len) // 128), self.MAX_SPLITS))
+        ctas = max(1, n_single * self.ctas_per_entry)
+        return max(1, min(self.slots // ctas, 7 * self.ctx.num_sms // (4 * ctas), -(-self._span(max_kv_len) // self.MIN_RANGE), self.ROWS_MAX_SPLITS))
 
-    def _rows_splits(self, n_single: int, max_kv_len: int) -> int:
-        ctas = max(1, n_single * self.ctas_per_tile)
-        return max(1, min(self.slots // ctas, -(-self._span(max_kv_len) // 128), self.ROWS_MAX_SPLITS))
+    def single_tokens(self, q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, block_table: torch.Tensor, cu_q: torch.Tensor,
+                      kv_len: torch.Tensor, entries: torch.Tensor, max_kv_len: int, scale: float, **opts) -> None:
+        """Attention of the entries that bring one token (in a bfloat16 engine)."""
+        splits = self.ranges(entries.numel(), max_kv_len)
+        if self.fast_single:
+            K.attention_single(q, out, kv, block_table, cu_q, kv_len, entries, self.Hq, self.Hkv, self.hd, scale, self.window,
+                               self.block, self.vd, splits=splits, part=self.part, maps=self.maps, value_in_key=self.value_in_key, **opts)
+        else:
+            K.attention_rows_single(q, out, kv, block_table, cu_q, kv_len, entries, self.zero_tok0[: entries.numel()], self.Hq,
+                                    self.Hkv, self.hd, scale, self.window, self.vd, splits=splits, part=self.part, maps=self.maps,
+                                    value_in_key=self.value_in_key, block=self.block, **opts)
 
     def __call__(self, q: torch.Tensor, out: torch.Tensor, step: StepContext, cache: PagedLayerCache, scale: float,
                  softcap: Optional[float] = None, sink_values: Optional[torch.Tensor] = None,
-                 slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 slopes: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+                 gate: Optional[torch.Tensor] = None, gate_scale: float = 1.0) -> torch.Tensor:
+        """`gate` (fp32 [T, heads]): the heads' outputs are multiplied by gate_scale * sigmoid(gate) before they are rounded."""
         g = step.groups[cache.group]
-        opts = dict(value_dim=self.vd, sink=sink_values is not None, softcap=softcap, sink_values=sink_values,
-                    maps=self.maps, value_in_key=self.value_in_key, slopes=slopes, bias=bias)
+        opts = dict(sink=sink_values is not None, softcap=softcap, sink_values=sink_values, slopes=slopes, bias=bias, gate=gate,
+                    gate_scale=gate_scale)
         if self._single is not None:
             (single,) = step.index(self._single)
-            if single.numel() and self.fast_single:
-                K.attention_single(q, out, cache.kv, g.block_table, step.cu_q, step.kv_len, single, self.Hq, self.Hkv,
-                                   self.hd, scale, self.window, self.block, splits=self._splits(single.numel(), step.max_kv_len),
-                                   part=self.part, **opts)
-            elif single.numel():
-                K.attention_rows(q, out, cache.kv, g.block_table, step.cu_q, step.kv_len, single,
-                                 self.zero_tok0[: single.numel()], self.Hq, self.Hkv, self.hd, scale, self.window,
-                                 splits=self._rows_splits(single.numel(), step.max_kv_len), part=self.part,
-                                 block=self.block, **opts)
+            if single.numel():
+                self.single_tokens(q, out, cache.kv, g.block_table, step.cu_q, step.kv_len, single, step.max_kv_len, scale, **opts)
+        opts.update(value_dim=self.vd, maps=self.maps, value_in_key=self.value_in_key)
         tile_entry, tile_tok0 = step.index(self._tiles)
         if tile_entry.numel():
             if self.rows:
@@ -363,12 +371,14 @@ class LatentAttention(Mixer):
         torch.bmm(q_plain.view(T, H, self.hd).transpose(0, 1), self.w_uk,
                   out=q_full.view(T, H, self.kd)[:, :, : self.rank].transpose(0, 1))
         lat = torch.empty((T, H * self.rank), dtype=dt, device=x.device)
-        self.attend(q_full, lat, step, cache, self.scale, sink_values=self.sink_values)
+        # a head's one factor passes through W_uv: the attention applies it to the head's weighted sum of latents
+        self.attend(q_full, lat, step, cache, self.scale, sink_values=self.sink_values,
+                    gate=proj[:, n_low: n_low + H] if self.gate == "head" else None)
         y = torch.empty((T, H * self.vd), dtype=dt, device=x.device)
         torch.bmm(lat.view(T, H, self.rank).transpose(0, 1), self.w_uv, out=y.view(T, H, self.vd).transpose(0, 1))
-        if self.gate:
+        if self.gate == "channel":
             gated = torch.empty_like(y)
-            K.sigmoid_gate(y, proj[:, n_low:], self.vd if self.gate == "head" else 1, gated)
+            K.sigmoid_gate(y, proj[:, n_low:], 1, gated)
             y = gated
         return self.o(y, out_dtype=torch.float32)
 
@@ -537,16 +547,9 @@ class DistanceBiasAttention(Mixer):
                       bool(pos and pos.layout == "interleaved"), g.slot_of_token if cache.writes else None,
                       cache.kv if cache.writes else None, q, self.H, self.G, self.hd, self.vd, True, conv=conv,
                       q_scale=self.temperature.factor if self.temperature else None)
-        if self.head_gate:
-            o = torch.empty((T, self.H * self.vd), dtype=torch.float32, device=x.device)
-            self.attend(q, o, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes,
-                        bias=self.bias_rows)
-            y = torch.empty((T, self.H * self.vd), dtype=dt, device=x.device)
-            K.sigmoid_gate(o, proj[:, nqkv:], self.vd, y, scale=out_scale)
-        else:
-            if out_scale != 1.0:
-                raise ValueError("a factor on the output rides on the heads' gate; this mixer has none")
-            y = torch.empty((T, self.H * self.vd), dtype=dt, device=x.device)
-            self.attend(q, y, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes,
-                        bias=self.bias_rows)
+        if out_scale != 1.0 and not self.head_gate:
+            raise ValueError("a factor on the output rides on the heads' gate; this mixer has none")
+        y = torch.empty((T, self.H * self.vd), dtype=dt, device=x.device)
+        self.attend(q, y, step, cache, self.scale, sink_values=self.sink_values, slopes=self.slopes, bias=self.bias_rows,
+                    gate=proj[:, nqkv: nqkv + self.H] if self.head_gate else None, gate_scale=out_scale)
         return project_out(self.o, y, add_to)

@@ -21,7 +21,7 @@ BF = torch.bfloat16
 # max |engine - plain| / max |plain| over the compared logits.  fp32 sums a few hundred products per output
 # against float64, and every sublayer's output is divided by its own root mean square before it is added (a small
 # output's rounding grows with it); in bfloat16 projections and activations are rounded to 8 bits.
-TOL = {"float32": 2e-5, "bfloat16": 4e-2}
+TOL = {"float32": 2e-5, "bfloat16": 6e-2}
 DTYPES = ["float32", "bfloat16"]
 NAMES = sorted(CONFIGS)
 
@@ -172,6 +172,82 @@ def test_latent_queries_alone(H, d, r, rank, dtype):
     want = torch.stack([a * cc - b * ss, b * cc + a * ss], dim=-1).reshape(T, H, r)
     got = qf.view(T, H, kd).double().cpu()
     assert rel_err(got[..., rank:], want) < tol and bool((got[..., :rank] == 7.0).all())
+
+
+@pytest.mark.parametrize("H,G,dk,dv,maps,vik", [(4, 2, 64, 64, 1, False), (8, 1, 16, 32, 1, False), (20, 1, 32, 16, 1, False), (6, 2, 48, 80, 1, False),
+                                               (12, 2, 16, 48, 2, False), (3, 3, 128, 128, 1, False), (12, 1, 96, 80, 1, True), (70, 1, 32, 16, 1, True),
+                                               (5, 1, 160, 128, 1, True), (40, 2, 16, 16, 1, False)])
+@pytest.mark.parametrize("page", [8, 16, 12])
+def test_single_tokens_on_the_tensor_cores(H, G, dk, dv, maps, vik, page):
+    """The kernel whose warps share the keys of one entry: groups of 1 to 70 heads, maps, values inside the keys, every option
+    of the scores, a gate; a far key and keys at the window's edges made to stand out; lengths of one key and more, in 1 to 7
+    ranges of which some are empty; pages scrambled, the rest poisoned; other entries of the batch untouched."""
+    lens = [1, 2, 33, 64, 257, 330]
+    per = G * (maps * dk + (0 if vik else dv))
+    blocks = -(-max(lens) // page)
+    tab = (torch.randperm(len(lens) * blocks, generator=torch.Generator().manual_seed(5)) + 1).view(len(lens), blocks)
+    keys = [torch.nn.functional.normalize(rnd(n, G * maps, dk, seed=10 + i), dim=-1) * 4.0 for i, n in enumerate(lens)]
+    keys = [k.to(BF).float() for k in keys]
+    vals = [k[:, :, :dv] if vik else rnd(n, G, dv, seed=30 + i).to(BF).float() for i, (n, k) in enumerate(zip(lens, keys))]
+    cache = torch.full((len(lens) * blocks + 1, page * per), 1e4)
+    for i, n in enumerate(lens):
+        for t in range(n):
+            row, off = cache[int(tab[i, t // page])], t % page
+            row[: G * maps * page * dk].view(G * maps, page, dk)[:, off] = keys[i][t]
+            if not vik:
+                row[G * maps * page * dk:].view(G, page, dv)[:, off] = vals[i][t]
+    plain = maps == 1 and dk == dv and not vik
+    dev_cache = cache.to(BF).to(DEV)
+    dev_cache = dev_cache.view(-1, 2, G, page, dk) if plain else dev_cache
+    Q = 2 + len(lens)                                             # two more tokens in front, of an entry that is not single
+    q, gate = rnd(Q, H, dk, seed=1), rnd(Q, H, seed=2)
+    sink, slopes, bias = rnd(H, seed=3) + 1.0, torch.rand(H, generator=torch.Generator().manual_seed(4)) / 20, rnd(H, 40, seed=5) * 2
+    per_head = H // (G * maps)
+    kh_of = [(h // maps) // per_head * maps + h % maps for h in range(H)]
+    vh_of = [(h // maps) // per_head for h in range(H)]
+    for opt in ("plain", "window", "block", "bias", "bias_window", "slopes", "cap"):
+        if vik and "bias" in opt:
+            continue
+        window = {"window": 37, "bias_window": 64}.get(opt)
+        block = 50 if opt == "block" else None
+        targets = [n - 1 if not window else max(0, n - window) for n in lens]       # the last key seen stands out
+        if not window and not block:
+            targets = [0] * len(lens)
+        for i, (n, tg) in enumerate(zip(lens, targets)):
+            for h in range(H):
+                k = keys[i][tg, kh_of[h]]
+                q[2 + i, h] = k * (0.75 + 0.02 * h / H)
+        qr = q.to(BF).float()
+        want = torch.empty(len(lens), H, dv, dtype=F64)
+        for i, n in enumerate(lens):
+            p = n - 1
+            j = torch.arange(n)
+            seen = (p - j < window) if window else torch.ones(n, dtype=torch.bool)
+            if block:
+                seen = seen & (j // block == p // block)
+            for h in range(H):
+                s = keys[i][:, kh_of[h]].to(F64) @ qr[2 + i, h].to(F64) * 0.9
+                if opt == "cap":
+                    s = 3.0 * torch.tanh(s / 3.0)
+                if opt == "slopes":
+                    s = s - slopes[h].to(F64) * (p - j)
+                if "bias" in opt:
+                    s = s + bias[h].to(F64)[(p - j).clamp(max=39)]
+                w = P.softmax_with_sink(s[None, None], seen[None], sink[h].to(F64)[None] if opt != "block" else None)[0, 0]
+                want[i, h] = (w @ vals[i][:, vh_of[h]].to(F64)) * torch.sigmoid(gate[2 + i, h].to(F64)) * 0.8
+        table = i32([[0] * blocks] + tab.tolist())
+        cu, kv = i32([0] + [2 + i for i in range(len(lens) + 1)]), i32([2] + lens)
+        entries, zeros = i32([-1] + list(range(1, len(lens) + 1))), i32([0] * 8)
+        for splits in (1, 2, 7):
+            out = torch.full((Q, H * dv), 55.0, device=DEV)
+            n = K().attention_rows_scratch_floats(entries.numel(), H, G, dv, maps, splits)
+            part = torch.full((max(1, n),), float("nan"), device=DEV)
+            K().attention_rows_single(qr.reshape(Q, -1).to(BF).to(DEV), out, dev_cache, table, cu, kv, entries, zeros, H, G, dk, 0.9, window, dv,
+                                      sink=opt != "block", softcap=3.0 if opt == "cap" else None, sink_values=sink.to(DEV) if opt != "block" else None,
+                                      maps=maps, value_in_key=vik, splits=splits, part=part, slopes=slopes.to(DEV) if opt == "slopes" else None,
+                                      bias=bias.to(DEV) if "bias" in opt else None, block=block, gate=gate.to(DEV), gate_scale=0.8)
+            assert float((out[2:].cpu().view(-1, H, dv).to(F64) - want).abs().max()) < 1e-4, (opt, splits)
+            assert bool((out[:2] == 55.0).all())
 
 
 # ================================================================================= mixers alone
