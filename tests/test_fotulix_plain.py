@@ -133,7 +133,7 @@ def test_layer_written_out():
 
 
 # --------------------------------------------------------------------- tables the package makes
-@pytest.mark.parametrize("dims,base,yarn", [(16, 500000.0, (4.0, 512, 32.0, 1.0)), (8, 3000.0, (3.0, 64, 8.0, 0.5)), (4, 40.0, (5.0, 30, 2.0, 1.0)),
+@pytest.mark.parametrize("dims,base,yarn", [(24, 70000.0, (6.0, 700, 24.0, 1.5)), (8, 3000.0, (3.0, 64, 8.0, 0.5)), (4, 40.0, (5.0, 30, 2.0, 1.0)),
                                             (64, 10000.0, (40.0, 4096, 32.0, 1.0)), (2, 10.0, (2.0, 16, 1.0, 1.0)), (12, 100.0, None)])
 def test_yarn_tables(dims, base, yarn):
     from rustinfer_b200.parts.rope import RotaryEncoding
@@ -149,7 +149,7 @@ def test_yarn_tables(dims, base, yarn):
     assert torch.allclose(c, torch.cos(ang) * mag, atol=1e-12) and torch.allclose(s, torch.sin(ang) * mag, atol=1e-12)
 
 
-@pytest.mark.parametrize("dims,base,bands", [(64, 20000.0, (4.0, 1.0, 4.0, 2048)), (8, 500.0, (4.0, 1.0, 4.0, 48)), (40, 70.0, (2.0, 2.0, 3.0, 20))])
+@pytest.mark.parametrize("dims,base,bands", [(48, 30000.0, (6.0, 1.5, 5.0, 1500)), (8, 500.0, (4.0, 1.0, 4.0, 48)), (40, 70.0, (2.0, 2.0, 3.0, 20))])
 def test_banded_tables(dims, base, bands):
     from rustinfer_b200.config.fotulix_config import BandScaling
     from rustinfer_b200.parts.rope import RotaryEncoding
@@ -159,7 +159,7 @@ def test_banded_tables(dims, base, bands):
     assert torch.allclose(c, torch.cos(ang), atol=1e-12) and torch.allclose(s, torch.sin(ang), atol=1e-12)
 
 
-@pytest.mark.parametrize("coef,every", [(0.5, 256), (1.5, 3), (0.0, 7), (-0.2, 1), (0.3, 2.5)])
+@pytest.mark.parametrize("coef,every", [(0.6, 200), (1.5, 3), (0.0, 7), (-0.2, 1), (0.3, 2.5)])
 def test_query_temperature_table(coef, every):
     from rustinfer_b200.parts.rope import QueryTemperature
     assert torch.allclose(QueryTemperature({"coef": coef, "every": every}).table(700), P.query_temperature(700, coef, every), atol=1e-14)
